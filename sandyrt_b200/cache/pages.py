@@ -110,7 +110,7 @@ class CacheLayout:
 
     @classmethod
     def _from_json(cls, j, specs=()) -> "CacheLayout":
-        groups = [CacheGroup(g["index"], PagedKVSpec(g["n_kv_heads"], g["head_dim"], g["window"] or None), list(g["caches"]))
+        groups = [CacheGroup(g["index"], PagedKVSpec(g["n_kv_heads"], g["head_dim"], g["window"] or None, g["keep_first"]), list(g["caches"]))
                   for g in j["groups"]]
         states = {}
         for ci in j["state_caches"]:

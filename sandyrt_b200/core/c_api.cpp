@@ -159,7 +159,8 @@ std::vector<CacheSpec> cache_specs_from(const Json& j) {
         if (s.is_null()) { out.push_back(CacheSpec::none()); continue; }
         const std::string kind = s.at("kind").as_string();
         if (kind == "paged") {
-            CacheSpec p = CacheSpec::paged((int)s.at("n_kv_heads").as_int(), (int)s.at("head_dim").as_int(), (int)geti(s, "window", 0));
+            CacheSpec p = CacheSpec::paged((int)s.at("n_kv_heads").as_int(), (int)s.at("head_dim").as_int(), (int)geti(s, "window", 0),
+                                           (int)geti(s, "keep_first", 0));
             p.planes = (int)geti(s, "planes", 2) == 1 ? 1 : 2;
             out.push_back(p);
         }
@@ -188,6 +189,7 @@ Json layout_json(const CacheLayout& l) {
         e["n_kv_heads"] = g.spec.n_kv_heads;
         e["head_dim"] = g.spec.head_dim;
         e["window"] = g.spec.window;
+        e["keep_first"] = g.spec.keep_first;
         e["planes"] = g.spec.planes;
         groups.push(e);
     }
@@ -590,6 +592,7 @@ Json call_model(Model& model, const std::string& m, const Json& a) {
                 e["n_kv_heads"] = c.n_kv_heads;
                 e["head_dim"] = c.head_dim;
                 e["window"] = c.window;
+                e["keep_first"] = c.keep_first;
                 e["planes"] = c.planes;
             }
             if (c.has_state()) {

@@ -11,12 +11,13 @@ namespace sandy {
 size_t dtype_size(DType d) { return d == DType::BF16 ? 2 : 4; }
 const char* dtype_name(DType d) { return d == DType::BF16 ? "bfloat16" : (d == DType::F32 ? "float32" : "int32"); }
 
-CacheSpec CacheSpec::paged(int n_kv_heads, int head_dim, int window) {
+CacheSpec CacheSpec::paged(int n_kv_heads, int head_dim, int window, int keep_first) {
     CacheSpec s;
     s.kind = Kind::PagedKV;
     s.n_kv_heads = n_kv_heads;
     s.head_dim = head_dim;
     s.window = window;
+    s.keep_first = window ? keep_first : 0;       // without a window everything stays anyway
     return s;
 }
 CacheSpec CacheSpec::paged_one_plane(int n_kv_heads, int head_dim, int window) {
@@ -40,12 +41,22 @@ CacheSpec CacheSpec::paged_with_state(int n_kv_heads, int head_dim, int window, 
 }
 CacheSpec CacheSpec::pages_only() const {
     if (!has_pages()) return none();
-    CacheSpec s = paged(n_kv_heads, head_dim, window);
+    CacheSpec s = paged(n_kv_heads, head_dim, window, keep_first);
     s.planes = planes;
     return s;
 }
+CacheSpec CacheSpec::shared(const CacheSpec& a, const CacheSpec& b) {
+    CacheSpec out = a, like_a = b;
+    like_a.window = a.window;
+    like_a.keep_first = a.keep_first;
+    if (like_a != a) throw CacheError("two layers of one cache entry have different needs");
+    if (!a.has_pages()) return out;
+    out.window = a.window && b.window ? std::max(a.window, b.window) : 0;
+    out.keep_first = out.window ? std::max(a.keep_first, b.keep_first) : 0;
+    return out;
+}
 bool CacheSpec::operator==(const CacheSpec& o) const {
-    return kind == o.kind && n_kv_heads == o.n_kv_heads && head_dim == o.head_dim && window == o.window && planes == o.planes &&
+    return kind == o.kind && n_kv_heads == o.n_kv_heads && head_dim == o.head_dim && window == o.window && keep_first == o.keep_first && planes == o.planes &&
            state_shape == o.state_shape && state_dtype == o.state_dtype;
 }
 
@@ -141,7 +152,7 @@ std::vector<RequestId> BlockAllocator::live() const {
     return out;
 }
 
-// Blocks below this index hold only positions no later query of a request of `length` tokens reads.
+// Blocks below this index hold only positions no later query of a request of `length` tokens reads (but for kept first ones).
 int BlockAllocator::first_needed_block(int group, int length) const {
     const int window = layout_.groups[(size_t)group].spec.window;
     if (!window) return 0;
@@ -214,12 +225,14 @@ void BlockAllocator::commit(RequestId rid, int new_len) {
     for (size_t g = 0; g < r.blocks.size(); g++) {
         auto& bl = r.blocks[g];
         const int first = std::min(first_needed_block((int)g, new_len), (int)bl.size());
+        const int keep = layout_.groups[g].spec.keep_first;
+        const int from = (keep + layout_.page_size - 1) / layout_.page_size;      // the blocks before stay with the request
         std::vector<int> gone;
-        for (int i = 0; i < first; i++)
+        for (int i = from; i < first; i++)
             if (bl[(size_t)i] != kFreed) gone.push_back(bl[(size_t)i]);
         if (!gone.empty()) {
             pools_[g].release(gone);
-            for (int i = 0; i < first; i++) bl[(size_t)i] = kFreed;
+            for (int i = from; i < first; i++) bl[(size_t)i] = kFreed;
             r.version = ++stamp_;
         }
     }

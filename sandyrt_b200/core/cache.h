@@ -13,7 +13,7 @@
 // be a run); many requests live at once and share the pools; a request has one block list per
 // *group* (all layers of a group use the same page ids), not one page table per tensor; pages of
 // a group whose layers only look back `window` positions are given back as soon as the window has
-// passed them; every request also holds one *state slot*, a row index into per-request state of
+// passed them (but for those of a sequence's first positions, where the layers keep them in sight); every request also holds one *state slot*, a row index into per-request state of
 // fixed size; and a page is an index into one arena per group, allocated once:
 // [caches in group][num_pages][K|V][Hkv][page_size][D] in the compute dtype.
 //
@@ -49,6 +49,7 @@ struct CacheSpec {
     // PagedKV: keys and values of every position (or of the last `window` positions) in pages
     int n_kv_heads = 0, head_dim = 0;
     int window = 0;                        // 0: all positions stay; n: only the last n are read
+    int keep_first = 0;                    // with a window: positions 0 .. keep_first - 1 stay as well
     // 2: a page holds keys and values; 1: one plane only, and a view's values are its keys' own numbers
     // (attention over a latent that is key and value at once: a head's output is then as wide as the keys
     // and the caller keeps the columns that mean something)
@@ -59,12 +60,15 @@ struct CacheSpec {
     DType state_dtype = DType::F32;
 
     static CacheSpec none() { return CacheSpec(); }
-    static CacheSpec paged(int n_kv_heads, int head_dim, int window = 0);
+    static CacheSpec paged(int n_kv_heads, int head_dim, int window = 0, int keep_first = 0);
     static CacheSpec paged_one_plane(int n_kv_heads, int head_dim, int window = 0);
     static CacheSpec state(std::vector<int64_t> shape, DType dtype = DType::F32);
     static CacheSpec paged_with_state(int n_kv_heads, int head_dim, int window, std::vector<int64_t> shape, DType dtype = DType::F32);
     bool has_pages() const { return kind == Kind::PagedKV || kind == Kind::PagedState; }
     bool has_state() const { return kind == Kind::State || kind == Kind::PagedState; }
+    // The needs of two layers that work on one cache entry (one reads what the other writes): pages stay as long as either
+    // still reads them.  CacheError if they differ in anything but their windows.
+    static CacheSpec shared(const CacheSpec& a, const CacheSpec& b);
     CacheSpec pages_only() const;          // what decides the page group: the state fields dropped
     bool operator==(const CacheSpec& o) const;
     bool operator!=(const CacheSpec& o) const { return !(*this == o); }

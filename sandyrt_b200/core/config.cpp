@@ -254,6 +254,15 @@ std::map<std::string, Architecture>& table() {
             return describe_tifepel(*g);
         };
         t[tifepel.name] = std::move(tifepel);
+        Architecture pugalix;
+        pugalix.name = PugalixConfig::kArchitecture;
+        pugalix.parse = [](const Json& raw) { return std::unique_ptr<ModelConfig>(new PugalixConfig(PugalixConfig::from_json(raw))); };
+        pugalix.describe = [](const ModelConfig& c) {
+            const auto* g = dynamic_cast<const PugalixConfig*>(&c);
+            if (!g) throw ConfigError("Pugalix was given another architecture's configuration");
+            return describe_pugalix(*g);
+        };
+        t[pugalix.name] = std::move(pugalix);
     });
     return t;
 }

@@ -170,6 +170,33 @@ public:
     void validate() const override;
 };
 
+// Pugalix's config.json (core/pugalix.cpp says what the keys mean): layers listed one by one, each a windowed attention
+// that keeps the first tokens in sight, a gated linear attention or a matrix memory; a dense feed-forward, or none.
+class PugalixConfig : public ModelConfig {
+public:
+    static constexpr const char* kArchitecture = "Pugalix";
+    struct Layer {
+        std::string type;                                   // "attention" | "gla" | "mlstm"
+        int64_t heads = 0, dim = 0, vdim = 0;
+        int64_t kv_heads = 0, rot_dims = 0;                 // attention (rot_dims 0: no rotary positions)
+        double scale = 1.0, rot_base = 10000.0;
+        int64_t window = 0, keep_first = 0;                 // attention (window 0: none)
+        int64_t kv_from = -1;                               // attention: >= 0: the layer whose keys and values it reads
+        double tau = 1.0;                                   // gla
+        int64_t rank = 0;                                   // gla: the decay's rank (0: the weight file's)
+        double gate_cap = 1.0;                              // mlstm
+        int64_t ff = 0;                                     // 0: the layer has no feed-forward
+    };
+    int64_t vocab = 0, width = 0;
+    double norm_eps = 1e-6, embedding_scale = 1.0;
+    std::vector<Layer> layers;
+
+    static PugalixConfig from_json(const Json& raw);
+    std::string architecture() const override { return kArchitecture; }
+    Json to_json() const override;
+    void validate() const override;
+};
+
 // A configuration of an architecture defined outside this library: its normalised config.json
 // as the architecture's own `parse` returned it.
 class ForeignConfig : public ModelConfig {
@@ -207,5 +234,6 @@ ModelSpec describe_panupel(const PanupelConfig& cfg);
 ModelSpec describe_sovezen(const SovezenConfig& cfg);
 ModelSpec describe_bilurax(const BiluraxConfig& cfg);
 ModelSpec describe_tifepel(const TifepelConfig& cfg);
+ModelSpec describe_pugalix(const PugalixConfig& cfg);
 
 }  // namespace sandy

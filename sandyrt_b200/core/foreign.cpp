@@ -51,7 +51,9 @@ public:
                     int window = 0;
                     if (const Json* w = c->find("window"))
                         if (!w->is_null()) window = (int)w->as_int();
-                    info_.cache = CacheSpec::paged((int)c->at("n_kv_heads").as_int(), (int)c->at("head_dim").as_int(), window);
+                    const Json* keep = c->find("keep_first");
+                    info_.cache = CacheSpec::paged((int)c->at("n_kv_heads").as_int(), (int)c->at("head_dim").as_int(), window,
+                                                   keep && !keep->is_null() ? (int)keep->as_int() : 0);
                 } else if (kind == "state") {
                     std::vector<int64_t> shape;
                     for (const Json& d : c->at("shape").items()) shape.push_back(d.as_int());

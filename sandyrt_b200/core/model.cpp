@@ -89,9 +89,15 @@ std::vector<CacheSpec> Model::cache_specs() const {
     std::vector<CacheSpec> specs((size_t)spec_.n_caches());
     std::vector<char> seen(specs.size(), 0);
     for (const LayerCall& c : spec_.schedule) {
-        const CacheSpec s = blocks_[(size_t)c.layer]->cache_spec();
-        if (seen[(size_t)c.cache] && specs[(size_t)c.cache] != s)
-            throw ConfigError("cache entry " + std::to_string(c.cache) + " is used by layers with different needs");
+        CacheSpec s = blocks_[(size_t)c.layer]->cache_spec();
+        if (seen[(size_t)c.cache]) {
+            // a layer that reads another's keys and values may look back less or further: the pages stay for both
+            try {
+                s = CacheSpec::shared(specs[(size_t)c.cache], s);
+            } catch (const CacheError&) {
+                throw ConfigError("cache entry " + std::to_string(c.cache) + " is used by layers with different needs");
+            }
+        }
         specs[(size_t)c.cache] = s;
         seen[(size_t)c.cache] = 1;
     }

@@ -489,6 +489,14 @@ void attention(const Launch& l, const AttentionStep& s, const Tensor& q, const K
     const int n_dist = extras ? extras->n_dist : 0;
     if (db && n_dist < 1) throw UnsupportedShape("attention: a bias by distance needs at least one row");
     const bool ruled = cap > 0.0f || chunk > 0;           // only kernels with a form for these rules take such steps
+    const int keep = extras && window > 0 ? extras->keep_first : 0;
+    const Tensor* eg = extras ? extras->elem_gate : nullptr;
+    if (keep < 0 || (keep > 0 && chunk > 0)) throw UnsupportedShape("attention: kept first keys go with a window and without chunks");
+    if (eg && (eg->dtype != q.dtype || eg->rows != q.rows || eg->cols % n_heads || eg->cols / n_heads > c.head_dim))
+        throw KernelError("attention: a gate by element is [T, H * dim] of the queries' type");
+    const bool gated = keep > 0 || eg;                    // likewise: the prompt kernels, mma.sync and heads-as-rows decode, general
+    const SandyAttentionRules rules = {window, keep, cap, chunk, sk, og, db, n_dist, eg ? eg->data : nullptr,
+                                       eg ? (int)eg->ld : 0, eg ? (int)(eg->cols / n_heads) : 0};
     const int d = c.head_dim, hkv = c.n_kv_heads;
     if (d % 16 != 0 || d > kMaxHeadDim) throw UnsupportedShape("attention: head size " + std::to_string(d) + " must be a multiple of 16, at most " + std::to_string(kMaxHeadDim));
     if (hkv <= 0 || n_heads % hkv != 0)
@@ -503,18 +511,18 @@ void attention(const Launch& l, const AttentionStep& s, const Tensor& q, const K
     if (s.max_q_len > 1 && q.dtype == DType::BF16 && d <= 128) {
         static const bool use_tc = env_int("SANDYRT_PREFILL_TC", 1) != 0;     // 0 keeps every head size on the mma.sync kernel
         if (use_tc && d == 64 && !db) {                       // (the tcgen05 kernel has no form for a bias by distance)
-            static auto fn = SANDY_KERNEL(attention_prefill_tc, sandy_prefill_attention_tc_cap);
+            static auto fn = SANDY_KERNEL(attention_prefill_tc, sandy_prefill_attention_tc_rules);
             OpTimer timer(l, "attention, prompt (tcgen05)", attn_bytes, attn_flops);
             const int code = fn(q.data, (int)q.ld, c.k, c.v, c.page_stride, s.block_table, s.max_blocks, s.q_start, s.kv_before,
-                                out.data, (int)out.ld, s.n_seqs, s.max_q_len, n_heads, hkv, d, c.page_size, scale, window,
-                                cap, chunk, c.num_pages, sk, og, l.kernel_status, l.stream);
+                                out.data, (int)out.ld, s.n_seqs, s.max_q_len, n_heads, hkv, d, c.page_size, scale, &rules,
+                                c.num_pages, l.kernel_status, l.stream);
             if (code != -1) { check(code, "prefill_attention_tc" + shape); return; }
         }
-        static auto fn = SANDY_KERNEL(attention_prefill, sandy_prefill_attention_bias);
+        static auto fn = SANDY_KERNEL(attention_prefill, sandy_prefill_attention_rules);
         OpTimer timer(l, "attention, prompt (mma.sync)", attn_bytes, attn_flops);
         check(fn(q.data, (int)q.ld, c.k, c.v, c.page_stride, s.block_table, s.max_blocks, s.q_start, s.kv_before, out.data,
-                 (int)out.ld, s.n_seqs, s.max_q_len, n_heads, hkv, d, c.page_size, scale, window, cap, chunk, c.num_pages, sk, og,
-                 db, n_dist, l.kernel_status, l.stream),
+                 (int)out.ld, s.n_seqs, s.max_q_len, n_heads, hkv, d, c.page_size, scale, &rules, c.num_pages, l.kernel_status,
+                 l.stream),
               "prefill_attention" + shape);
         return;
     }
@@ -527,24 +535,25 @@ void attention(const Launch& l, const AttentionStep& s, const Tensor& q, const K
     // 8 x 392: 9.4 / 8.7; 8 tokens x 24 heads x 392: 11.3 / 16.6; 8 x 12 x 2,000: 13.2 / 36.2.
     // Steps with capped scores, chunks of positions or a bias by distance: this kernel is the decode kernel that has a form
     // for them, so it takes them all (with few keys it is one launch of one split); a chunk bounds the keys a query walks.
+    // Steps with kept first keys or a gate by element: heads of 64 may also take the mma.sync kernel further down.
+    const int seen_keys = window > 0 ? std::min(window + keep, s.max_blocks * c.page_size) : s.max_blocks * c.page_size;
     if (s.max_q_len == 1 && q.dtype == DType::BF16 && d <= 128 && T <= 65535 &&
-        (ruled || db || (n_heads / hkv >= kSharedKvMinHeads && (int64_t)T * n_heads * s.max_blocks * c.page_size >= kSharedKvMinTriples))) {
-        const int max_kv = chunk > 0 ? std::min(chunk, s.max_blocks * c.page_size) : s.max_blocks * c.page_size;
+        (ruled || db || (gated && d != 64) || (n_heads / hkv >= kSharedKvMinHeads && (int64_t)T * n_heads * s.max_blocks * c.page_size >= kSharedKvMinTriples))) {
+        const int max_kv = chunk > 0 ? std::min(chunk, seen_keys) : seen_keys;
         const int tiles = hkv * ((n_heads / hkv + 15) / 16), groups = (max_kv + 15) / 16;
         const int splits = std::max(1, std::min({(groups + 3) / 4, (2 * sm_count() + T * tiles - 1) / (T * tiles), 64}));
         static auto need = SANDY_KERNEL(attention_decode_shared, sandy_decode_attention_shared_scratch);
-        static auto fn = SANDY_KERNEL(attention_decode_shared, sandy_decode_attention_shared_bias);
+        static auto fn = SANDY_KERNEL(attention_decode_shared, sandy_decode_attention_shared_rules);
         const long long floats = need(T, n_heads, hkv, d, splits);
         float* scratch = floats ? (float*)ws.raw("decode_attention_partial_rows", (size_t)floats * sizeof(float)) : nullptr;
         OpTimer timer(l, "attention, decode (heads as rows)", attn_bytes, attn_flops);
         check(fn(q.data, (int)q.ld, c.k, c.v, c.page_stride, s.block_table, s.max_blocks, s.token_seq, s.positions, out.data, (int)out.ld,
-                 T, n_heads, hkv, d, c.page_size, scale, window, cap, chunk, splits, c.num_pages, sk, og, db, n_dist, scratch,
-                 l.kernel_status, l.stream),
+                 T, n_heads, hkv, d, c.page_size, scale, &rules, splits, c.num_pages, scratch, l.kernel_status, l.stream),
               "decode_attention_shared" + shape);
         return;
     }
     if (!db && !ruled && s.max_q_len == 1 && decode_head_dim(q.dtype, d)) {
-        const int max_kv = s.max_blocks * c.page_size;
+        const int max_kv = seen_keys;
         const int splits = std::min(decode_splits(T, n_heads, max_kv), kClusterMaxSplits);
         const size_t stage = 2 * (size_t)c.page_size * (size_t)d * q.elem_size();
         const bool fits = stage * 4 <= 160 * 1024;           // the ring holds at least four stages
@@ -556,19 +565,21 @@ void attention(const Launch& l, const AttentionStep& s, const Tensor& q, const K
         // 8 tokens of 1,000 keys 12.9 / 12.5 / 7.8.  So it takes every launch but those with so many pairs that
         // a pair is one block (one split), where the bulk kernel's deeper ring of pages keeps its small lead.
         static const int mma_mode = env_int("SANDYRT_DECODE_MMA", 1);          // 0 keeps the two kernels below, for comparisons
-        if (mma_mode != 0 && q.dtype == DType::BF16 && d == 64 && !(bulk && splits == 1)) {
+        if (q.dtype == DType::BF16 && d == 64 && (gated || (mma_mode != 0 && !(bulk && splits == 1)))) {
             static auto max_keys_fn = SANDY_KERNEL(attention_decode_mma, sandy_decode_attention_mma_max_keys);
             if (max_kv <= max_keys_fn(splits, c.page_size)) {
-                static auto fn = SANDY_KERNEL(attention_decode_mma, sandy_decode_attention_mma_ext);
+                static auto fn = SANDY_KERNEL(attention_decode_mma, sandy_decode_attention_mma_rules);
                 OpTimer timer(l, "attention, decode (mma.sync)", attn_bytes, attn_flops);
                 check(fn(q.data, (int)q.ld, c.k, c.v, c.page_stride, s.block_table, s.max_blocks, s.token_seq, s.positions, out.data,
-                         (int)out.ld, T, n_heads, hkv, d, c.page_size, scale, window, splits, c.num_pages, max_kv, sk, og, l.kernel_status,
+                         (int)out.ld, T, n_heads, hkv, d, c.page_size, scale, &rules, splits, c.num_pages, max_kv, l.kernel_status,
                          l.stream),
                       "decode_attention_mma" + shape);
                 return;
             }
         }
-        if (bulk) {
+        if (gated) {
+            // no form here: the general kernel below
+        } else if (bulk) {
             static auto fn = SANDY_KERNEL(attention_decode_bulk, sandy_decode_attention_bulk_ext);
             OpTimer timer(l, "attention, decode (bulk copies)", attn_bytes, attn_flops);
             check(fn(q.data, (int)q.ld, c.k, c.v, c.page_stride, s.block_table, s.max_blocks, s.token_seq, s.positions, out.data,
@@ -590,13 +601,12 @@ void attention(const Launch& l, const AttentionStep& s, const Tensor& q, const K
                      sk, og, l.kernel_status, l.stream),
                   "decode_attention" + shape);
         }
-        return;
+        if (!gated) return;
     }
-    static auto fn = SANDY_KERNEL(attention, sandy_paged_attention_bias);
+    static auto fn = SANDY_KERNEL(attention, sandy_paged_attention_rules);
     OpTimer timer(l, "attention, general", attn_bytes, attn_flops);
     check(fn(q.data, (int)q.ld, c.k, c.v, c.page_stride, s.block_table, s.max_blocks, s.token_seq, s.positions, out.data,
-             (int)out.ld, T, n_heads, hkv, d, c.page_size, scale, window, cap, chunk, c.num_pages, code_of(q.dtype), sk, og, db,
-             n_dist, l.kernel_status, l.stream),
+             (int)out.ld, T, n_heads, hkv, d, c.page_size, scale, &rules, c.num_pages, code_of(q.dtype), l.kernel_status, l.stream),
           "paged_attention" + shape);
 }
 
@@ -880,13 +890,13 @@ void attention_prepare(const Launch& l, const AttentionPrepare& p, const Tensor&
     if (proj.dtype != c.dtype || q_out.dtype != proj.dtype || q_out.rows != proj.rows || q_out.cols != (int64_t)p.n_heads * c.head_dim ||
         c.n_kv_heads != p.n_kv_heads || c.head_dim < p.qk_dim || c.head_dim < p.v_dim)
         throw KernelError("attention_prepare: the projection, the queries and the cache disagree");
-    static auto fn = SANDY_KERNEL(attention_prepare, sandy_attention_prepare_pos);
+    static auto fn = SANDY_KERNEL(attention_prepare, sandy_attention_prepare_rot);
     OpTimer timer(l, "q/k norm + rotary + cache write", 2.0 * tensor_bytes(&proj), 0);
     check(fn(proj.data, (int)proj.ld, p.q_off, p.k_off, p.v_off, (int)proj.rows, p.n_heads, p.n_kv_heads, p.qk_dim, p.v_dim,
              c.head_dim, p.q_gain, p.k_gain, p.eps, p.freq, p.rot_dims, positions, token_seq, block_table, max_blocks, c.k, c.v,
              c.page_stride, c.page_size, c.num_pages, p.write_cache ? 1 : 0, q_out.data, (int)q_out.ld, p.gate_in, p.ld_gate,
              p.gate_out, p.gate_scale, p.q_head_scale, p.v_unit_eps, p.per_head_norm ? 1 : 0, p.q_pos_coef, p.q_pos_every,
-             code_of(proj.dtype), l.kernel_status, l.stream),
+             p.interleaved ? 1 : 0, code_of(proj.dtype), l.kernel_status, l.stream),
           "attention_prepare");
 }
 
@@ -1100,6 +1110,36 @@ void mlstm_scan(const Launch& l, const StepSeqs& s, const MlstmShape& m, const T
                       gate_bias, m.cap, m.q_scale, (float*)state.data, state.row_elems, s.q_start, s.seq_slots, (float*)out.data,
                       (int)out.ld, s.n_seqs, m.n_heads, m.qk_dim, m.v_dim, long_from, l.stream),
               "mlstm_chunk_scan" + shape);
+}
+
+int64_t gla_state_floats(const GlaShape& m) { return (int64_t)m.n_heads * m.v_dim * m.qk_dim; }
+
+void gla_scan(const Launch& l, const StepSeqs& s, const GlaShape& m, const Tensor& proj, const Tensor& low, const Tensor& w2t,
+              const Tensor& bias, const StateView& state, Tensor& out, int max_q_len, Workspace& ws) {
+    const int64_t HD = (int64_t)m.n_heads * m.qk_dim;
+    if (out.dtype != DType::F32 || out.cols != (int64_t)m.n_heads * m.v_dim || low.dtype != DType::F32 || w2t.dtype != DType::F32 ||
+        w2t.rows != low.cols || w2t.cols != HD || !w2t.contiguous() || bias.dtype != DType::F32 || bias.numel() != HD ||
+        state.dtype != DType::F32 || state.row_elems < gla_state_floats(m) || proj.rows != s.n_tokens || low.rows != s.n_tokens)
+        throw KernelError("gla_scan: shapes disagree");
+    static auto fn = SANDY_KERNEL(gated_linear, sandy_gla_scan);
+    static auto chunked = SANDY_KERNEL(gated_linear, sandy_gla_chunk_scan);
+    static auto need = SANDY_KERNEL(gated_linear, sandy_gla_scratch_floats);
+    const int long_from = max_q_len >= kChunkedFrom ? kChunkedFrom : 0;
+    const double st = 2.0 * s.n_seqs * m.n_heads * m.qk_dim * m.v_dim * 4.0;
+    const std::string shape = "(d=" + std::to_string(m.qk_dim) + ",e=" + std::to_string(m.v_dim) + ")";
+    float* scratch = long_from ? (float*)ws.raw("gla_chunks", (size_t)need(s.n_tokens, s.n_seqs, m.n_heads, m.qk_dim) * sizeof(float)) : nullptr;
+    OpTimer timer(l, "gated linear attention: recurrence", st + tensor_bytes(&out), 4.0 * s.n_tokens * m.n_heads * m.qk_dim * m.v_dim);
+    check(fn(proj.data, (int)proj.ld, code_of(proj.dtype), m.q_off, m.k_off, m.v_off, (const float*)low.data, (int)low.ld, (int)low.cols,
+             (const float*)w2t.data, (const float*)bias.data, m.inv_tau, m.q_scale, (float*)state.data, state.row_elems, s.q_start,
+             s.seq_slots, (float*)out.data, (int)out.ld, s.n_seqs, m.n_heads, m.qk_dim, m.v_dim, long_from, l.stream),
+          "gla_scan" + shape);
+    if (!long_from) return;
+    g_launches++;                                          // two launches
+    check(chunked(proj.data, (int)proj.ld, code_of(proj.dtype), m.q_off, m.k_off, m.v_off, (const float*)low.data, (int)low.ld, (int)low.cols,
+                  (const float*)w2t.data, (const float*)bias.data, m.inv_tau, m.q_scale, (float*)state.data, state.row_elems, s.q_start,
+                  s.seq_slots, (float*)out.data, (int)out.ld, scratch, s.n_tokens, s.n_seqs, max_q_len, m.n_heads, m.qk_dim, m.v_dim,
+                  long_from, l.stream),
+          "gla_chunk_scan" + shape);
 }
 
 void sample(const Launch& l, const Tensor& logits, int* out_tokens, const float* temperature, const int* top_k,

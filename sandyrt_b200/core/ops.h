@@ -142,6 +142,11 @@ struct AttentionExtras {
     // the score of query i and key j after the scale and the cap.  Null: none.
     const float* dist_bias = nullptr;
     int n_dist = 0;
+    // With a window: the sequence's first keys that stay visible behind it (not together with chunks).
+    int keep_first = 0;
+    // A gate by element: entry i of head h's output is multiplied by sigmoid(elem_gate[t, h * dim + i]), dim the head's share
+    // of the gate's columns (entries from dim on are padding).  Pre-activations of q's type; null: none.
+    const Tensor* elem_gate = nullptr;
 };
 // The widest head any attention kernel takes (the general kernel; the tensor-core prompt kernels take up to 128, the
 // decode kernels 16 / 32 / 64 / 128 and, in bfloat16, 256).
@@ -280,6 +285,7 @@ struct AttentionPrepare {
                                                                    // the gains may then be null
     float q_pos_coef = 0.0f;                                       // with q_pos_every > 0 the query at position p is multiplied by
     int q_pos_every = 0;                                           // 1 + q_pos_coef * ln(floor((p + 1) / q_pos_every) + 1)
+    bool interleaved = false;                                      // the rotation pairs 2i with 2i + 1 (else i with i + rot_dims / 2)
     bool write_cache = true;
 };
 void attention_prepare(const Launch& l, const AttentionPrepare& p, const Tensor& proj, const KVView& cache,
@@ -310,6 +316,17 @@ struct MlstmShape { int n_heads = 0, qk_dim = 0, v_dim = 0, q_off = 0, k_off = 0
 // gates float32 [T, >= 2H]: input-gate pre-activations, then forget-gate ones; gate_bias float32 [2H].
 void mlstm_scan(const Launch& l, const StepSeqs& s, const MlstmShape& m, const Tensor& proj, const Tensor& gates,
                 const float* gate_bias, const StateView& state, Tensor& out, int max_q_len);
+
+// ---- gated linear attention: a decay per key channel and token (gated_linear.cu) --------------------------------
+struct GlaShape {
+    int n_heads = 0, qk_dim = 0, v_dim = 0, q_off = 0, k_off = 0, v_off = 0;      // columns of q, k, v in the projection
+    float inv_tau = 1.0f, q_scale = 1.0f;
+};
+int64_t gla_state_floats(const GlaShape& m);                       // S [H][v_dim][qk_dim]
+// S_t = diag(alpha_t) S_(t-1) + k_t v_t^T, out_t = S_t^T (q_t q_scale); alpha = sigmoid(low w2t + bias)^inv_tau per key channel.
+// low float32 [T, rank]; w2t float32 [rank, H * qk_dim]; bias float32 [H * qk_dim]; out float32 [T, H * v_dim].
+void gla_scan(const Launch& l, const StepSeqs& s, const GlaShape& m, const Tensor& proj, const Tensor& low, const Tensor& w2t,
+              const Tensor& bias, const StateView& state, Tensor& out, int max_q_len, Workspace& ws);
 
 // The last n_taps - 1 rows of `rows` ([T, channels], any pitch) of every request into its state at tail_off, as the
 // convolutions above keep theirs (rows before the step come from the old tail).

@@ -429,6 +429,7 @@ Table& table() {
             register_latent_parts();
             register_capped_parts();
             register_stream_parts();
+            register_linear_parts();
         });
         entered = false;
     }

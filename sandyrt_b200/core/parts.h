@@ -295,6 +295,10 @@ void register_latent_parts();
 // with a learned bias by distance, and the state-space mixer with one decay per head.
 void register_stream_parts();
 
+// Kinds of parts_linear.cpp: attention with a sliding window that keeps the first tokens, a one in the softmax's
+// denominator and a gate by element; gated linear attention; the matrix memory as a mixer of its own.
+void register_linear_parts();
+
 template <typename T>
 std::unique_ptr<T> make_part(const std::string& family, const PartSpec& spec) {
     std::unique_ptr<Part> p = get_part(family, spec.kind).make(spec);

@@ -30,7 +30,8 @@ int Scheduler::pages_for(int group, int n_tokens) const {
     if (window) {
         // pages covering the window plus the portion being appended
         const int span = std::min(n_tokens, window + opt_.prefill_chunk);
-        return std::min(all, (span + ps - 1) / ps + 1);
+        const int kept = (alloc_.layout().groups[(size_t)group].spec.keep_first + ps - 1) / ps;
+        return std::min(all, (span + ps - 1) / ps + 1 + kept);
     }
     return all;
 }

@@ -28,6 +28,10 @@
 // This is the general kernel: any head size that is a multiple of 16 up to 640 (two instantiations: up to
 // 256, and beyond for the wide rows of attention over a latent), any number of heads and groups, both
 // storage types.  One warp owns one (token, head) pair.
+//
+// A window may leave the sequence's first keys visible (keep_first: attention with kept first tokens), and a head's output
+// may be multiplied element by element with the sigmoid of a gate (attention_rules.h).
+#include "attention_rules.h"
 #include "common.cuh"
 
 namespace {
@@ -107,7 +111,8 @@ paged_attention_kernel(const T* __restrict__ q, int ld_q,
                        int n_tokens, int n_heads, int n_kv_heads, int head_dim, int page_size,
                        float scale, int window, float softcap, int chunk, int num_pages,
                        const float* __restrict__ sink, const float* __restrict__ out_gate,
-                       const float* __restrict__ dist_bias, int n_dist, int* __restrict__ status) {
+                       const float* __restrict__ dist_bias, int n_dist, int keep_first, const T* __restrict__ elem_gate,
+                       int ld_elem_gate, int gate_dim, int* __restrict__ status) {
     __shared__ float q_smem[WARPS_PER_BLOCK][MAX_D];
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const long long pair = (long long)blockIdx.x * WARPS_PER_BLOCK + warp;
@@ -116,8 +121,7 @@ paged_attention_kernel(const T* __restrict__ q, int ld_q,
     const int s = token_seq[t];
     const int pos = positions[t];
     const int kvh = h / (n_heads / n_kv_heads);
-    int lo = window > 0 ? max(0, pos + 1 - window) : 0;
-    if (chunk > 0) lo = max(lo, pos - pos % chunk);
+    const VisibleKeys seen = visible_keys(pos, window, keep_first, chunk);
     const int* table = block_table + (size_t)s * max_blocks;
     const long long rows_per_page = page_stride / head_dim;  // page stride in rows of D
 
@@ -130,9 +134,9 @@ paged_attention_kernel(const T* __restrict__ q, int ld_q,
 #pragma unroll
     for (int i = 0; i < MAX_D / 32; i++) acc[i] = 0.0f;
 
-    for (int base = lo; base <= pos; base += 32) {
-        const int j = base + lane;
-        const bool valid = j <= pos;
+    for (int base = 0; base < seen.n; base += 32) {
+        const bool valid = base + lane < seen.n;
+        const int j = seen.position(base + lane);
         long long row = 0;  // row index (units of D elements) of key j inside the layer's cache
         float sc = -INFINITY;
         if (valid) {
@@ -153,7 +157,7 @@ paged_attention_kernel(const T* __restrict__ q, int ld_q,
         l = l * corr + warp_sum(p);
 #pragma unroll
         for (int i = 0; i < MAX_D / 32; i++) acc[i] *= corr;
-        const int count = min(32, pos - base + 1);
+        const int count = min(32, seen.n - base);
         for (int jj = 0; jj < count; jj++) {
             const float pj = __shfl_sync(0xffffffffu, p, jj);
             const long long rj = __shfl_sync(0xffffffffu, row, jj);
@@ -172,7 +176,8 @@ paged_attention_kernel(const T* __restrict__ q, int ld_q,
 #pragma unroll
     for (int i = 0; i < MAX_D / 32; i++) {
         const int d = lane + 32 * i;
-        if (d < head_dim) out[(size_t)t * ld_out + h * head_dim + d] = from_f32<T>(acc[i] * inv);
+        if (d < head_dim)
+            out[(size_t)t * ld_out + h * head_dim + d] = from_f32<T>(acc[i] * inv * elem_gate_of(elem_gate, ld_elem_gate, gate_dim, t, h, d));
     }
 }
 
@@ -210,16 +215,22 @@ SANDY_API int sandy_kv_append(const void* k_src, const void* v_src, int ld_src,
 // denominator.  out_gate: float32 [n_tokens, H] or null: a factor on each head's output.
 // out_gate: float32 [n_tokens, H] or null: a factor on each head's output.  softcap 0: scores as they are; chunk 0: no chunks.
 // dist_bias: float32 [H, n_dist] or null: entry min(i - j, n_dist - 1) of the head's row is added to the score of query i
-// and key j (after the scale and the cap), a learned bias by distance.
-SANDY_API int sandy_paged_attention_bias(const void* q, int ld_q, const void* k_cache, const void* v_cache,
-                                         long long page_stride, const int* block_table, int max_blocks,
-                                         const int* token_seq, const int* positions, void* out, int ld_out,
-                                         int n_tokens, int n_heads, int n_kv_heads, int head_dim, int page_size,
-                                         float scale, int window, float softcap, int chunk, int num_pages, int dtype,
-                                         const float* sink, const float* out_gate, const float* dist_bias, int n_dist,
-                                         int* status, cudaStream_t stream) {
+// and key j (after the scale and the cap), a learned bias by distance.  rules->keep_first and rules->elem_gate as in
+// attention_rules.h.
+SANDY_API int sandy_paged_attention_rules(const void* q, int ld_q, const void* k_cache, const void* v_cache,
+                                          long long page_stride, const int* block_table, int max_blocks,
+                                          const int* token_seq, const int* positions, void* out, int ld_out,
+                                          int n_tokens, int n_heads, int n_kv_heads, int head_dim, int page_size,
+                                          float scale, const SandyAttentionRules* rules, int num_pages, int dtype,
+                                          int* status, cudaStream_t stream) {
     if (n_tokens == 0) return SANDY_OK;
+    if (!rules) return SANDY_ERR_ARGUMENT;
+    const int window = rules->window, chunk = rules->chunk, n_dist = rules->n_dist;
+    const float softcap = rules->softcap;
+    const float *sink = rules->sink, *out_gate = rules->out_gate, *dist_bias = rules->dist_bias;
     if (dist_bias && n_dist < 1) return SANDY_ERR_ARGUMENT;
+    if (rules->keep_first < 0 || (rules->keep_first > 0 && chunk > 0) || (rules->elem_gate && rules->gate_dim < 1))
+        return SANDY_ERR_UNSUPPORTED;
     if (!q || !k_cache || !v_cache || !block_table || !token_seq || !positions || !out)
         return SANDY_ERR_ARGUMENT;
     if (head_dim <= 0 || head_dim % 16 != 0 || head_dim > WIDE_HEAD_DIM) return SANDY_ERR_UNSUPPORTED;
@@ -231,12 +242,27 @@ SANDY_API int sandy_paged_attention_bias(const void* q, int ld_q, const void* k_
     (head_dim <= MAX_HEAD_DIM ? paged_attention_kernel<T, MAX_HEAD_DIM> : paged_attention_kernel<T, WIDE_HEAD_DIM>)<<<blocks, WARPS_PER_BLOCK * 32, 0, stream>>>( \
         (const T*)q, ld_q, (const T*)k_cache, (const T*)v_cache, page_stride, block_table, max_blocks, \
         token_seq, positions, (T*)out, ld_out, n_tokens, n_heads, n_kv_heads, head_dim, page_size,    \
-        scale, window, softcap, chunk, num_pages, sink, out_gate, dist_bias, n_dist, status)
+        scale, window, softcap, chunk, num_pages, sink, out_gate, dist_bias, n_dist, rules->keep_first,   \
+        (const T*)rules->elem_gate, rules->ld_elem_gate, rules->gate_dim, status)
     if (dtype == SANDY_F32) LAUNCH(float);
     else if (dtype == SANDY_BF16) LAUNCH(bf16);
     else return SANDY_ERR_UNSUPPORTED;
 #undef LAUNCH
     return sandy_launch_status();
+}
+
+// The same without kept first keys or a gate by element.
+SANDY_API int sandy_paged_attention_bias(const void* q, int ld_q, const void* k_cache, const void* v_cache,
+                                         long long page_stride, const int* block_table, int max_blocks,
+                                         const int* token_seq, const int* positions, void* out, int ld_out,
+                                         int n_tokens, int n_heads, int n_kv_heads, int head_dim, int page_size,
+                                         float scale, int window, float softcap, int chunk, int num_pages, int dtype,
+                                         const float* sink, const float* out_gate, const float* dist_bias, int n_dist,
+                                         int* status, cudaStream_t stream) {
+    const SandyAttentionRules rules = {window, 0, softcap, chunk, sink, out_gate, dist_bias, n_dist, nullptr, 0, 0};
+    return sandy_paged_attention_rules(q, ld_q, k_cache, v_cache, page_stride, block_table, max_blocks, token_seq, positions, out,
+                                       ld_out, n_tokens, n_heads, n_kv_heads, head_dim, page_size, scale, &rules, num_pages, dtype,
+                                       status, stream);
 }
 
 // The same without a bias by distance.

@@ -24,11 +24,13 @@
 // Rows of keys outside the range (or without a page) are zero-filled in shared memory, so that a
 // poisoned slot never meets a zero of P.  As in attention_decode.cu the first groups -- all positions but the token's own, which
 // the kernel before is still writing -- are asked for BEFORE the wait on that kernel, and up to 8
-// splits of a pair merge as one thread-block cluster through distributed shared memory.
+// splits of a pair merge as one thread-block cluster through distributed shared memory.  With kept first keys behind a
+// window (keep_first) the visible keys are numbered through, the kept ones first, and the splits cut those numbers.
 // Softmax statistics and the accumulator are float; P is rounded to bfloat16 for the product (the
 // row sum is taken before rounding).
 #include <cooperative_groups.h>
 
+#include "attention_rules.h"
 #include "common.cuh"
 
 namespace cg = cooperative_groups;
@@ -74,9 +76,10 @@ __device__ __forceinline__ uint32_t pack_bf16(float lo, float hi) {
 // The last step of a softmax row (maxima here are in units of log 2): a sink joins the denominator, nothing in the
 // numerator; an output gate scales the head's result.
 __device__ __forceinline__ float finish_row2(float O, float L, float M, const float* sink, const float* out_gate, int t,
-                                             int h, int n_heads) {
+                                             int h, int n_heads, const bf16* elem_gate, int ld_elem_gate, int gate_dim, int d) {
     if (sink && M > -INFINITY) L += exp2f(sink[h] * 1.4426950408889634f - M);
-    const float g = out_gate ? out_gate[(size_t)t * n_heads + h] : 1.0f;
+    float g = out_gate ? out_gate[(size_t)t * n_heads + h] : 1.0f;
+    g *= elem_gate_of(elem_gate, ld_elem_gate, gate_dim, t, h, d);
     return L > 0.0f ? O / L * g : 0.0f;
 }
 
@@ -86,7 +89,8 @@ decode_attention_mma_kernel(const bf16* __restrict__ q, int ld_q, const bf16* __
                             int max_blocks, const int* __restrict__ token_seq, const int* __restrict__ positions,
                             bf16* __restrict__ out, int ld_out, int n_heads, int n_kv_heads, int page_size, float scale,
                             int window, int num_splits, int num_pages, const float* __restrict__ sink,
-                            const float* __restrict__ out_gate, int* __restrict__ status) {
+                            const float* __restrict__ out_gate, int keep_first, const bf16* __restrict__ elem_gate,
+                            int ld_elem_gate, int gate_dim, int* __restrict__ status) {
     // a warp's own stages: [stage][keys | values][16 rows of 128 bytes]
     __shared__ __align__(128) uint8_t st[WARPS][STAGES][2][GROUP_BYTES];
     __shared__ int s_pages[MAX_PAGES];
@@ -105,20 +109,25 @@ decode_attention_mma_kernel(const bf16* __restrict__ q, int ld_q, const bf16* __
     const int s = token_seq[t];
     const int pos = positions[t];
     const int kvh = h / (n_heads / n_kv_heads);
-    const int lo = window > 0 ? max(0, pos + 1 - window) : 0;
-    const int n_keys = pos - lo + 1;
+    const VisibleKeys seen = visible_keys(pos, window, keep_first, 0);
+    const int n_keys = seen.n;
     int chunk = (n_keys + num_splits - 1) / num_splits;
     chunk = (chunk + GROUP - 1) / GROUP * GROUP;
-    const int begin = lo + split * chunk;
-    const int end = min(pos + 1, begin + chunk);
+    const int begin = split * chunk;                        // [begin, end): numbers of visible keys
+    const int end = min(n_keys, begin + chunk);
     const int n_groups = end > begin ? (end - begin + GROUP - 1) / GROUP : 0;          // groups of 16 keys
     const int my_groups = n_groups > warp ? (n_groups - warp + WARPS - 1) / WARPS : 0;  // this warp takes groups warp, warp + 4, ..
     const int* table = block_table + (size_t)s * max_blocks;
 
-    // the pages of the block's range, once
-    const int p0 = begin / page_size;
-    const int n_pages = end > begin ? (end - 1) / page_size - p0 + 1 : 0;
-    for (int i = tid; i < n_pages && i < MAX_PAGES; i += WARPS * 32) s_pages[i] = p0 + i < max_blocks ? table[p0 + i] : -1;
+    // the pages of the block's range, once: those of its kept keys, then those of its keys in the window
+    const int kept_end = min(end, seen.kept);
+    const int kept_p0 = begin / page_size, kept_pages = kept_end > begin ? (kept_end - 1) / page_size - kept_p0 + 1 : 0;
+    const int p0 = seen.position(max(begin, seen.kept)) / page_size - kept_pages;      // a key's block minus this is its place
+    const int n_pages = end > max(begin, seen.kept) ? seen.position(end - 1) / page_size - p0 + 1 : kept_pages;
+    for (int i = tid; i < n_pages && i < MAX_PAGES; i += WARPS * 32) {
+        const int b = i < kept_pages ? kept_p0 + i : p0 + i;
+        s_pages[i] = b < max_blocks ? table[b] : -1;
+    }
     __syncthreads();
 
     // Copies this warp's k-th group of keys into its stage k % STAGES.  Keys at or past `end`, the key `skip`
@@ -132,14 +141,15 @@ decode_attention_mma_kernel(const bf16* __restrict__ q, int ld_q, const bf16* __
 #pragma unroll
         for (int i = 0; i < GROUP / 4; i++) {
             const int row = (lane >> 3) + 4 * i;
-            const int j = first + row;
+            const int v = first + row;
+            const int j = seen.position(v);
             const uint32_t at = row * 128 + ((c ^ (row & 7)) << 4);
-            bool ok = j < end && j != skip;
+            bool ok = v < end && j != skip;
             size_t off = 0;
             if (ok) {
                 const int blk = page_shift >= 0 ? j >> page_shift : j / page_size;
                 const int slot = page_shift >= 0 ? j & (page_size - 1) : j % page_size;
-                const int pi = blk - p0;
+                const int pi = blk - (v < seen.kept ? kept_p0 : p0);
                 const int page = pi < MAX_PAGES ? s_pages[pi] : -1;
                 if (page < 0 || page >= num_pages) {
                     if (status && c == 0) atomicOr(status, 16);     // a visible key with no page behind it
@@ -176,10 +186,10 @@ decode_attention_mma_kernel(const bf16* __restrict__ q, int ld_q, const bf16* __
         }
     }
     // the token's own key, if it lies in a group this warp staged without it
-    if (pos >= begin && pos < end) {
-        const int gi = (pos - begin) / GROUP;                 // its group in the block; this warp's k-th if gi = warp + 4 k
+    if (n_keys - 1 >= begin && n_keys - 1 < end) {            // the last visible key
+        const int gi = (n_keys - 1 - begin) / GROUP;                 // its group in the block; this warp's k-th if gi = warp + 4 k
         if (gi % WARPS == warp && gi / WARPS < pre && lane < 16) {
-            const int k = gi / WARPS, row = (pos - begin) % GROUP, is_v = lane / 8, c = lane % 8;
+            const int k = gi / WARPS, row = (n_keys - 1 - begin) % GROUP, is_v = lane / 8, c = lane % 8;
             const int pi = pos / page_size - p0;
             const int page = pi < MAX_PAGES ? s_pages[pi] : -1;
             if (page >= 0 && page < num_pages) {
@@ -301,7 +311,7 @@ decode_attention_mma_kernel(const bf16* __restrict__ q, int ld_q, const bf16* __
             }
         }
         if (!in_cluster) {
-            out[(size_t)t * ld_out + h * D + d] = __float2bfloat16_rn(finish_row2(O, L, M, sink, out_gate, t, h, n_heads));
+            out[(size_t)t * ld_out + h * D + d] = __float2bfloat16_rn(finish_row2(O, L, M, sink, out_gate, t, h, n_heads, elem_gate, ld_elem_gate, gate_dim, d));
         } else {
             first_all[split * (D + 2) + d] = O;
             if (d == 0) {
@@ -327,7 +337,7 @@ decode_attention_mma_kernel(const bf16* __restrict__ q, int ld_q, const bf16* __
                         O = fmaf(cl_all[r][d], w, O);
                     }
                 }
-                out[(size_t)t * ld_out + h * D + d] = __float2bfloat16_rn(finish_row2(O, L, M, sink, out_gate, t, h, n_heads));
+                out[(size_t)t * ld_out + h * D + d] = __float2bfloat16_rn(finish_row2(O, L, M, sink, out_gate, t, h, n_heads, elem_gate, ld_elem_gate, gate_dim, d));
             }
         }
     }
@@ -338,19 +348,24 @@ decode_attention_mma_kernel(const bf16* __restrict__ q, int ld_q, const bf16* __
 // Most keys a (token, head) pair may have with this many splits: a block keeps the page numbers of its range.
 SANDY_API int sandy_decode_attention_mma_max_keys(int num_splits, int page_size) {
     if (num_splits < 1 || page_size < 1) return 0;
-    const long long keys = (long long)(MAX_PAGES - 2) * page_size * num_splits;
+    const long long keys = (long long)(MAX_PAGES - 4) * page_size * num_splits;      // a range of kept keys and one of a window: two pages each for the ends
     return keys > 0x3fffffff ? 0x3fffffff : (int)keys;
 }
 
 // Arguments as sandy_decode_attention_cluster (attention_decode.cu); bfloat16, heads of 64, 1 <= num_splits <= 8;
 // max_keys: the longest visible range of any token of the launch (checked against the block's table of pages).
-SANDY_API int sandy_decode_attention_mma_ext(const void* q, int ld_q, const void* k_cache, const void* v_cache,
+// No form for capped scores, chunks of positions or a bias by distance.
+SANDY_API int sandy_decode_attention_mma_rules(const void* q, int ld_q, const void* k_cache, const void* v_cache,
                                              long long page_stride, const int* block_table, int max_blocks,
                                              const int* token_seq, const int* positions, void* out, int ld_out, int n_tokens,
                                              int n_heads, int n_kv_heads, int head_dim, int page_size, float scale,
-                                             int window, int num_splits, int num_pages, int max_keys, const float* sink,
-                                             const float* out_gate, int* status, cudaStream_t stream) {
+                                             const SandyAttentionRules* rules, int num_splits, int num_pages, int max_keys,
+                                             int* status, cudaStream_t stream) {
     if (n_tokens == 0) return SANDY_OK;
+    if (!rules) return SANDY_ERR_ARGUMENT;
+    if (rules->softcap != 0.0f || rules->chunk || rules->dist_bias || rules->keep_first < 0 || (rules->elem_gate && rules->gate_dim < 1))
+        return SANDY_ERR_UNSUPPORTED;
+    const int window = rules->window;
     if (!q || !k_cache || !v_cache || !block_table || !token_seq || !positions || !out) return SANDY_ERR_ARGUMENT;
     if (head_dim != D || num_splits < 1 || num_splits > MAX_CLUSTER_SPLITS) return SANDY_ERR_UNSUPPORTED;
     if (n_kv_heads <= 0 || n_heads % n_kv_heads != 0 || page_size <= 0 || window < 0) return SANDY_ERR_UNSUPPORTED;
@@ -383,8 +398,22 @@ SANDY_API int sandy_decode_attention_mma_ext(const void* q, int ld_q, const void
     const cudaError_t e = cudaLaunchKernelEx(&cfg, decode_attention_mma_kernel, (const bf16*)q, ld_q, (const bf16*)k_cache,
                                              (const bf16*)v_cache, page_stride, block_table, max_blocks, token_seq, positions,
                                              (bf16*)out, ld_out, n_heads, n_kv_heads, page_size, scale, window, num_splits,
-                                             num_pages, sink, out_gate, status);
+                                             num_pages, rules->sink, rules->out_gate, rules->keep_first,
+                                             (const bf16*)rules->elem_gate, rules->ld_elem_gate, rules->gate_dim, status);
     return e != cudaSuccess ? (int)e : (int)cudaGetLastError();
+}
+
+// The same without kept first keys or a gate by element.
+SANDY_API int sandy_decode_attention_mma_ext(const void* q, int ld_q, const void* k_cache, const void* v_cache,
+                                             long long page_stride, const int* block_table, int max_blocks,
+                                             const int* token_seq, const int* positions, void* out, int ld_out, int n_tokens,
+                                             int n_heads, int n_kv_heads, int head_dim, int page_size, float scale,
+                                             int window, int num_splits, int num_pages, int max_keys, const float* sink,
+                                             const float* out_gate, int* status, cudaStream_t stream) {
+    const SandyAttentionRules rules = {window, 0, 0.0f, 0, sink, out_gate, nullptr, 0, nullptr, 0, 0};
+    return sandy_decode_attention_mma_rules(q, ld_q, k_cache, v_cache, page_stride, block_table, max_blocks, token_seq, positions,
+                                            out, ld_out, n_tokens, n_heads, n_kv_heads, head_dim, page_size, scale, &rules,
+                                            num_splits, num_pages, max_keys, status, stream);
 }
 
 // The same without a sink or an output gate.

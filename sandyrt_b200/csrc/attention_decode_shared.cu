@@ -18,6 +18,8 @@
 // with more, every block leaves its partial rows in a scratch and a second kernel adds them in the splits' order.
 // Formula, sink and output factor as in attention.cu; scores, softmax and sums in 32-bit, base 2 exponentials, P
 // rounded to bfloat16 for the product (the row sum is taken before rounding).  Head sizes: multiples of 16 up to 128.
+// With kept first keys behind a window (keep_first) the visible keys are numbered through: the kept ones, then the window's.
+#include "attention_rules.h"
 #include "common.cuh"
 
 namespace {
@@ -69,7 +71,8 @@ decode_shared_kernel(const bf16* __restrict__ q, int ld_q, const bf16* __restric
                      const int* __restrict__ token_seq, const int* __restrict__ positions, bf16* __restrict__ out, int ld_out,
                      int n_heads, int n_kv_heads, int page_size, float scale, int window, float softcap, int chunk, int splits,
                      int num_pages, const float* __restrict__ sink, const float* __restrict__ out_gate,
-                     const float* __restrict__ dist_bias, int n_dist, float* __restrict__ scratch, int* __restrict__ status) {
+                     const float* __restrict__ dist_bias, int n_dist, int keep_first, const bf16* __restrict__ elem_gate,
+                     int ld_elem_gate, int gate_dim, float* __restrict__ scratch, int* __restrict__ status) {
     constexpr int PITCH = D + 8;                       // elements: ldmatrix rows fall on different banks
     constexpr int PIECES = D / 8;                      // 16-byte pieces of a key row
     extern __shared__ __align__(16) unsigned char smem_raw[];
@@ -87,9 +90,8 @@ decode_shared_kernel(const bf16* __restrict__ q, int ld_q, const bf16* __restric
     pdl_launch_dependents();
     const int pos = positions[t];
     const int* table = block_table + (size_t)token_seq[t] * max_blocks;
-    int lo = window > 0 ? max(0, pos + 1 - window) : 0;
-    if (chunk > 0) lo = max(lo, pos - pos % chunk);          // a query sees the keys of its own chunk of positions
-    const int n_groups = (pos + 1 - lo + GROUP - 1) / GROUP;
+    const VisibleKeys seen = visible_keys(pos, window, keep_first, chunk);
+    const int n_groups = (seen.n + GROUP - 1) / GROUP;
     const int per_split = (n_groups + splits - 1) / splits;
     const int g_begin = split * per_split, g_end = min(n_groups, g_begin + per_split);
 
@@ -111,7 +113,7 @@ decode_shared_kernel(const bf16* __restrict__ q, int ld_q, const bf16* __restric
             const int c = lane + 32 * i;
             if (c < GROUP * PIECES) {
                 const int r = c / PIECES, piece = c % PIECES;
-                const int key = lo + g * GROUP + r;
+                const int key = seen.position(g * GROUP + r);
                 long long src = -1;
                 if (key <= pos && key / page_size < max_blocks) {
                     const int page = table[key / page_size];
@@ -156,12 +158,11 @@ decode_shared_kernel(const bf16* __restrict__ q, int ld_q, const bf16* __restric
             mma16816(s[1], qa[kk], b[2], b[3]);
         }
         // s[nt][0..1]: row gq, keys nt * 8 + tq * 2 (+ 1); s[nt][2..3]: row gq + 8
-        const int key0 = lo + g * GROUP;
 #pragma unroll
         for (int nt = 0; nt < 2; nt++)
 #pragma unroll
             for (int j = 0; j < 4; j++) {
-                const int key = key0 + nt * 8 + tq * 2 + (j & 1);
+                const int key = seen.position(g * GROUP + nt * 8 + tq * 2 + (j & 1));
                 float sc = softcap > 0.0f ? cap2 * tanh_fast(s[nt][j] * over_cap) : s[nt][j] * s2;
                 if (dist_bias) {                               // a learned bias by distance, this row's head
                     const int hd = min(first_head + gq + (j >> 1) * 8, n_heads - 1);
@@ -246,6 +247,7 @@ decode_shared_kernel(const bf16* __restrict__ q, int ld_q, const bf16* __restric
             }
             float v = den > 0.0f ? num / den : 0.0f;
             if (out_gate) v *= out_gate[(size_t)t * n_heads + head];
+            v *= elem_gate_of(elem_gate, ld_elem_gate, gate_dim, t, head, col);
             out[(size_t)t * ld_out + (size_t)head * D + col] = __float2bfloat16_rn(v);
         }
     }
@@ -257,7 +259,8 @@ decode_shared_kernel(const bf16* __restrict__ q, int ld_q, const bf16* __restric
 template <int D>
 __global__ void __launch_bounds__(128)
 decode_shared_merge_kernel(const float* __restrict__ scratch, int splits, bf16* __restrict__ out, int ld_out, int n_heads,
-                           int n_kv_heads, const float* __restrict__ sink, const float* __restrict__ out_gate) {
+                           int n_kv_heads, const float* __restrict__ sink, const float* __restrict__ out_gate,
+                           const bf16* __restrict__ elem_gate, int ld_elem_gate, int gate_dim) {
     pdl_wait();
     pdl_launch_dependents();
     const int t = blockIdx.y;
@@ -289,6 +292,7 @@ decode_shared_merge_kernel(const float* __restrict__ scratch, int splits, bf16* 
     }
     float v = den > 0.0f ? num / den : 0.0f;
     if (out_gate) v *= out_gate[(size_t)t * n_heads + head];
+    v *= elem_gate_of(elem_gate, ld_elem_gate, gate_dim, t, head, col);
     out[(size_t)t * ld_out + (size_t)head * D + col] = __float2bfloat16_rn(v);
 }
 
@@ -302,8 +306,7 @@ size_t smem_bytes(bool one_plane) {
 template <int D>
 int launch(const bf16* q, int ld_q, const bf16* k, const bf16* v, long long page_stride, const int* block_table, int max_blocks,
            const int* token_seq, const int* positions, bf16* out, int ld_out, int n_tokens, int n_heads, int n_kv_heads, int page_size,
-           float scale, int window, float softcap, int chunk, int splits, int num_pages, const float* sink, const float* out_gate,
-           const float* dist_bias, int n_dist, float* scratch, int* status, cudaStream_t stream) {
+           float scale, const SandyAttentionRules& r, int splits, int num_pages, float* scratch, int* status, cudaStream_t stream) {
     static bool configured = false;
     const size_t smem = smem_bytes<D>(k == v);
     if (!configured) {
@@ -314,11 +317,11 @@ int launch(const bf16* q, int ld_q, const bf16* k, const bf16* v, long long page
     const int group_heads = n_heads / n_kv_heads, tiles = n_kv_heads * ((group_heads + ROWS - 1) / ROWS);
     int code = sandy_launch(decode_shared_kernel<D>, dim3(splits, tiles, n_tokens), dim3(WARPS * 32), smem, stream, q, ld_q, k, v,
                             page_stride, block_table, max_blocks, token_seq, positions, out, ld_out, n_heads, n_kv_heads, page_size,
-                            scale, window, softcap, chunk, splits, num_pages, sink, out_gate, dist_bias, n_dist,
-                            splits > 1 ? scratch : (float*)nullptr, status);
+                            scale, r.window, r.softcap, r.chunk, splits, num_pages, r.sink, r.out_gate, r.dist_bias, r.n_dist,
+                            r.keep_first, (const bf16*)r.elem_gate, r.ld_elem_gate, r.gate_dim, splits > 1 ? scratch : (float*)nullptr, status);
     if (code != SANDY_OK || splits == 1) return code;
     return sandy_launch(decode_shared_merge_kernel<D>, dim3(tiles, n_tokens, (ROWS * D + 127) / 128), dim3(128), 0, stream, (const float*)scratch, splits, out,
-                        ld_out, n_heads, n_kv_heads, sink, out_gate);
+                        ld_out, n_heads, n_kv_heads, r.sink, r.out_gate, (const bf16*)r.elem_gate, r.ld_elem_gate, r.gate_dim);
 }
 
 }  // namespace
@@ -336,14 +339,19 @@ SANDY_API long long sandy_decode_attention_shared_scratch(int n_tokens, int n_he
 // floats as sandy_decode_attention_shared_scratch says (may be null with one split).  softcap > 0: a score becomes
 // softcap * tanh(score / softcap); chunk > 0: a query sees only keys j >= pos - pos % chunk.
 // dist_bias: float32 [n_heads, n_dist] or null: entry min(pos - j, n_dist - 1) of the head's row joins the score of key j.
-SANDY_API int sandy_decode_attention_shared_bias(const void* q, int ld_q, const void* k_cache, const void* v_cache, long long page_stride,
+// rules->keep_first and rules->elem_gate as in attention_rules.h.
+SANDY_API int sandy_decode_attention_shared_rules(const void* q, int ld_q, const void* k_cache, const void* v_cache, long long page_stride,
                                             const int* block_table, int max_blocks, const int* token_seq, const int* positions,
                                             void* out, int ld_out, int n_tokens, int n_heads, int n_kv_heads, int head_dim,
-                                            int page_size, float scale, int window, float softcap, int chunk, int splits,
-                                            int num_pages, const float* sink, const float* out_gate, const float* dist_bias,
-                                            int n_dist, float* scratch, int* status, cudaStream_t stream) {
+                                            int page_size, float scale, const SandyAttentionRules* rules, int splits,
+                                            int num_pages, float* scratch, int* status, cudaStream_t stream) {
     if (n_tokens == 0) return SANDY_OK;
-    if (dist_bias && n_dist < 1) return SANDY_ERR_ARGUMENT;
+    if (!rules) return SANDY_ERR_ARGUMENT;
+    const int window = rules->window, chunk = rules->chunk;
+    const float softcap = rules->softcap;
+    if (rules->dist_bias && rules->n_dist < 1) return SANDY_ERR_ARGUMENT;
+    if (rules->keep_first < 0 || (rules->keep_first > 0 && chunk > 0) || (rules->elem_gate && rules->gate_dim < 1))
+        return SANDY_ERR_UNSUPPORTED;
     if (!q || !k_cache || !v_cache || !block_table || !token_seq || !positions || !out) return SANDY_ERR_ARGUMENT;
     if (n_kv_heads <= 0 || n_heads % n_kv_heads || page_size <= 0 || window < 0 || splits < 1 || splits > 65535 ||
         n_tokens > 65535 || (splits > 1 && !scratch) || softcap < 0.0f || chunk < 0)
@@ -354,13 +362,26 @@ SANDY_API int sandy_decode_attention_shared_bias(const void* q, int ld_q, const 
 #define SANDY_CASE(DD)                                                                                                              \
     case DD:                                                                                                                        \
         return launch<DD>((const bf16*)q, ld_q, (const bf16*)k_cache, (const bf16*)v_cache, page_stride, block_table, max_blocks,  \
-                          token_seq, positions, (bf16*)out, ld_out, n_tokens, n_heads, n_kv_heads, page_size, scale, window, softcap, \
-                          chunk, splits, num_pages, sink, out_gate, dist_bias, n_dist, scratch, status, stream)
+                          token_seq, positions, (bf16*)out, ld_out, n_tokens, n_heads, n_kv_heads, page_size, scale, *rules, \
+                          splits, num_pages, scratch, status, stream)
     switch (head_dim) {
         SANDY_CASE(16); SANDY_CASE(32); SANDY_CASE(48); SANDY_CASE(64); SANDY_CASE(80); SANDY_CASE(96); SANDY_CASE(112); SANDY_CASE(128);
     }
 #undef SANDY_CASE
     return SANDY_ERR_UNSUPPORTED;
+}
+
+// The same without kept first keys or a gate by element.
+SANDY_API int sandy_decode_attention_shared_bias(const void* q, int ld_q, const void* k_cache, const void* v_cache, long long page_stride,
+                                            const int* block_table, int max_blocks, const int* token_seq, const int* positions,
+                                            void* out, int ld_out, int n_tokens, int n_heads, int n_kv_heads, int head_dim,
+                                            int page_size, float scale, int window, float softcap, int chunk, int splits,
+                                            int num_pages, const float* sink, const float* out_gate, const float* dist_bias,
+                                            int n_dist, float* scratch, int* status, cudaStream_t stream) {
+    const SandyAttentionRules rules = {window, 0, softcap, chunk, sink, out_gate, dist_bias, n_dist, nullptr, 0, 0};
+    return sandy_decode_attention_shared_rules(q, ld_q, k_cache, v_cache, page_stride, block_table, max_blocks, token_seq, positions,
+                                               out, ld_out, n_tokens, n_heads, n_kv_heads, head_dim, page_size, scale, &rules, splits,
+                                               num_pages, scratch, status, stream);
 }
 
 // The same without a bias by distance.

@@ -24,6 +24,10 @@
 //
 // P is rounded to bfloat16 for the P.V product (the row sum is taken before rounding).
 // Head sizes: multiples of 16 up to 128.  Larger heads, and float32, use the general kernel.
+//
+// With kept first keys behind a window (keep_first) the tiles of those keys come first and the tiles between them and
+// the window are left out.
+#include "attention_rules.h"
 #include "common.cuh"
 
 namespace {
@@ -83,7 +87,8 @@ prefill_attention_kernel(const bf16* __restrict__ q, int ld_q, const bf16* __res
                          const int* __restrict__ kv_before, bf16* __restrict__ out, int ld_out, int n_heads,
                          int n_kv_heads, int page_size, float scale, int window, float softcap, int chunk, int num_pages,
                          const float* __restrict__ sink, const float* __restrict__ out_gate,
-                         const float* __restrict__ dist_bias, int n_dist, int* __restrict__ status) {
+                         const float* __restrict__ dist_bias, int n_dist, int keep_first,
+                         const bf16* __restrict__ elem_gate, int ld_elem_gate, int gate_dim, int* __restrict__ status) {
     constexpr int LDS = D + 8;               // row pitch in elements: 16 bytes of padding
     constexpr int CHUNKS = D / 8;            // 16-byte pieces per row
     constexpr int KSTEPS = D / 16;           // k-steps of Q.K^T
@@ -111,7 +116,11 @@ prefill_attention_kernel(const bf16* __restrict__ q, int ld_q, const bf16* __res
     // the first key any row of the block sees: the window's edge and the start of the first row's chunk of positions
     int key_lo = window > 0 ? max(0, pos_first + 1 - window) : 0;
     if (chunk > 0) key_lo = max(key_lo, pos_first - pos_first % chunk);
-    const int kt_begin = key_lo / BN, kt_end = pos_last / BN;
+    const int kt_window = key_lo / BN, kt_end = pos_last / BN;
+    // kept first keys: their tiles, as far as the window does not hold them anyway, come in front of the window's
+    const int kept_tiles = window > 0 ? min((keep_first + BN - 1) / BN, kt_window) : 0;
+    const int n_it = kept_tiles + kt_end - kt_window + 1;
+    auto tile_at = [&](int it) { return it < kept_tiles ? it : it - kept_tiles + kt_window; };
     const int kvh = h / (n_heads / n_kv_heads);
     const int* table = block_table + (size_t)s * max_blocks;
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
@@ -144,7 +153,7 @@ prefill_attention_kernel(const bf16* __restrict__ q, int ld_q, const bf16* __res
                 const int page = b < max_blocks ? (table_staged ? s_table[b] : table[b]) : -1;
                 if (page < 0 || page >= num_pages) {
                     // a key with no page behind it; inside the visible range this is a fault
-                    if (j >= key_lo && status && c == 0) atomicOr(status, 16);
+                    if ((j >= key_lo || j < keep_first) && status && c == 0) atomicOr(status, 16);
                     ok = false;
                 } else {
                     off = (size_t)page * page_stride + ((size_t)kvh * page_size + (j & page_mask)) * D + c * 8;
@@ -154,9 +163,9 @@ prefill_attention_kernel(const bf16* __restrict__ q, int ld_q, const bf16* __res
             if (!one_plane) cp_async16(dv + r * LDS + c * 8, v_cache + off, ok ? 16 : 0);
         }
     };
-    load_kv(kt_begin, 0);
+    load_kv(tile_at(0), 0);
     cp_async_commit();
-    if (kt_begin < kt_end) load_kv(kt_begin + 1, 1);
+    if (n_it > 1) load_kv(tile_at(1), 1);
     cp_async_commit();
 
     float o[DTILES][4];
@@ -183,11 +192,12 @@ prefill_attention_kernel(const bf16* __restrict__ q, int ld_q, const bf16* __res
     uint32_t qa[KSTEPS][4];
     bool q_loaded = false;
 
-    for (int kt = kt_begin; kt <= kt_end; kt++) {
-        const int buf = (kt - kt_begin) % STAGES;
+    for (int it = 0; it < n_it; it++) {
+        const int kt = tile_at(it);
+        const int buf = it % STAGES;
         cp_async_wait<1>();          // tile kt has landed (tile kt+1 may still be on its way)
         __syncthreads();             // ... for everyone; and everyone is done with tile kt-1
-        if (kt + 2 <= kt_end) load_kv(kt + 2, (kt + 2 - kt_begin) % STAGES);     // into tile kt-1's buffer
+        if (it + 2 < n_it) load_kv(tile_at(it + 2), (it + 2) % STAGES);     // into the buffer of the tile before
         cp_async_commit();
         if (!q_loaded) {
 #pragma unroll
@@ -248,16 +258,16 @@ prefill_attention_kernel(const bf16* __restrict__ q, int ld_q, const bf16* __res
 #pragma unroll
                 for (int e = 0; e < 2; e++) {
                     const int j = j0 + e;
-                    if (!(j <= pos0 && j >= lo0)) sc[nt][e] = -INFINITY;
-                    if (!(j <= pos1 && j >= lo1)) sc[nt][2 + e] = -INFINITY;
+                    if (!(j <= pos0 && (j >= lo0 || j < keep_first))) sc[nt][e] = -INFINITY;
+                    if (!(j <= pos1 && (j >= lo1 || j < keep_first))) sc[nt][2 + e] = -INFINITY;
                 }
             } else {
                 const int j0 = kt * BN + khalf * BNW + nt * 8 + 2 * t;
 #pragma unroll
                 for (int e = 0; e < 2; e++) {
                     const int j = j0 + e;
-                    sc[nt][e] = (j <= pos0 && j >= lo0) ? sc[nt][e] * scale_log2 : -INFINITY;
-                    sc[nt][2 + e] = (j <= pos1 && j >= lo1) ? sc[nt][2 + e] * scale_log2 : -INFINITY;
+                    sc[nt][e] = (j <= pos0 && (j >= lo0 || j < keep_first)) ? sc[nt][e] * scale_log2 : -INFINITY;
+                    sc[nt][2 + e] = (j <= pos1 && (j >= lo1 || j < keep_first)) ? sc[nt][2 + e] * scale_log2 : -INFINITY;
                 }
             }
             m_new[0] = fmaxf(m_new[0], fmaxf(sc[nt][0], sc[nt][1]));
@@ -361,6 +371,14 @@ prefill_attention_kernel(const bf16* __restrict__ q, int ld_q, const bf16* __res
 #pragma unroll
     for (int dt = 0; dt < DTILES; dt++) {
         const int col = h * D + dt * 8 + 2 * t;
+        if (elem_gate) {
+#pragma unroll
+            for (int e = 0; e < 2; e++) {
+                const int i = dt * 8 + 2 * t + e;
+                if (row0 < rows_valid) o[dt][e] *= elem_gate_of(elem_gate, ld_elem_gate, gate_dim, qs + t0 + row0, h, i);
+                if (row1 < rows_valid) o[dt][2 + e] *= elem_gate_of(elem_gate, ld_elem_gate, gate_dim, qs + t0 + row1, h, i);
+            }
+        }
         if (row0 < rows_valid)
             *reinterpret_cast<uint32_t*>(out + (size_t)(qs + t0 + row0) * ld_out + col) =
                 pack_bf16(o[dt][0] * inv0, o[dt][1] * inv0);
@@ -373,9 +391,8 @@ prefill_attention_kernel(const bf16* __restrict__ q, int ld_q, const bf16* __res
 template <int D>
 int launch(const void* q, int ld_q, const void* k_cache, const void* v_cache, long long page_stride,
            const int* block_table, int max_blocks, const int* q_start, const int* kv_before, void* out, int ld_out,
-           int n_seqs, int max_q_len, int n_heads, int n_kv_heads, int page_size, float scale, int window, float softcap,
-           int chunk, int num_pages, const float* sink, const float* out_gate, const float* dist_bias, int n_dist, int* status,
-           cudaStream_t stream) {
+           int n_seqs, int max_q_len, int n_heads, int n_kv_heads, int page_size, float scale,
+           const SandyAttentionRules& r, int num_pages, int* status, cudaStream_t stream) {
     constexpr int LDS = D + 8;
     const int smem_two = (BM + 2 * STAGES * BN) * LDS * (int)sizeof(bf16);
     const int smem = k_cache == v_cache ? (BM + STAGES * BN) * LDS * (int)sizeof(bf16) : smem_two;
@@ -388,8 +405,8 @@ int launch(const void* q, int ld_q, const void* k_cache, const void* v_cache, lo
     dim3 grid((max_q_len + BM - 1) / BM, n_heads, n_seqs);
     prefill_attention_kernel<D><<<grid, THREADS, smem, stream>>>(
         (const bf16*)q, ld_q, (const bf16*)k_cache, (const bf16*)v_cache, page_stride, block_table, max_blocks, q_start,
-        kv_before, (bf16*)out, ld_out, n_heads, n_kv_heads, page_size, scale, window, softcap, chunk, num_pages, sink, out_gate,
-        dist_bias, n_dist, status);
+        kv_before, (bf16*)out, ld_out, n_heads, n_kv_heads, page_size, scale, r.window, r.softcap, r.chunk, num_pages, r.sink,
+        r.out_gate, r.dist_bias, r.n_dist, r.keep_first, (const bf16*)r.elem_gate, r.ld_elem_gate, r.gate_dim, status);
     return sandy_launch_status();
 }
 
@@ -399,15 +416,19 @@ int launch(const void* q, int ld_q, const void* k_cache, const void* v_cache, lo
 // kv_before: int32 [n_seqs], tokens each request had in the cache before the step;
 // max_q_len: the longest portion (sizes the grid).  Caches, sink, out_gate, softcap, chunk and dist_bias ([H, n_dist], a
 // learned bias by distance) as in attention.cu.
-SANDY_API int sandy_prefill_attention_bias(const void* q, int ld_q, const void* k_cache, const void* v_cache,
+SANDY_API int sandy_prefill_attention_rules(const void* q, int ld_q, const void* k_cache, const void* v_cache,
                                       long long page_stride, const int* block_table, int max_blocks,
                                       const int* q_start, const int* kv_before, void* out, int ld_out, int n_seqs,
                                       int max_q_len, int n_heads, int n_kv_heads, int head_dim, int page_size,
-                                      float scale, int window, float softcap, int chunk, int num_pages, const float* sink,
-                                      const float* out_gate, const float* dist_bias, int n_dist, int* status,
+                                      float scale, const SandyAttentionRules* rules, int num_pages, int* status,
                                       cudaStream_t stream) {
     if (n_seqs == 0 || max_q_len == 0) return SANDY_OK;
-    if (dist_bias && n_dist < 1) return SANDY_ERR_ARGUMENT;
+    if (!rules) return SANDY_ERR_ARGUMENT;
+    const int window = rules->window, chunk = rules->chunk;
+    const float softcap = rules->softcap;
+    if (rules->dist_bias && rules->n_dist < 1) return SANDY_ERR_ARGUMENT;
+    if (rules->keep_first < 0 || (rules->keep_first > 0 && chunk > 0) || (rules->elem_gate && rules->gate_dim < 1))
+        return SANDY_ERR_UNSUPPORTED;
     if (!q || !k_cache || !v_cache || !block_table || !q_start || !kv_before || !out) return SANDY_ERR_ARGUMENT;
     if (n_kv_heads <= 0 || n_heads % n_kv_heads != 0 || page_size <= 0 || window < 0 || softcap < 0.0f || chunk < 0)
         return SANDY_ERR_UNSUPPORTED;
@@ -420,11 +441,25 @@ SANDY_API int sandy_prefill_attention_bias(const void* q, int ld_q, const void* 
 #define CASE(DD)                                                                                                \
     if (head_dim == DD)                                                                                         \
         return launch<DD>(q, ld_q, k_cache, v_cache, page_stride, block_table, max_blocks, q_start, kv_before,  \
-                          out, ld_out, n_seqs, max_q_len, n_heads, n_kv_heads, page_size, scale, window,        \
-                          softcap, chunk, num_pages, sink, out_gate, dist_bias, n_dist, status, stream)
+                          out, ld_out, n_seqs, max_q_len, n_heads, n_kv_heads, page_size, scale, *rules,        \
+                          num_pages, status, stream)
     CASE(16); CASE(32); CASE(48); CASE(64); CASE(80); CASE(96); CASE(112); CASE(128);
 #undef CASE
     return SANDY_ERR_UNSUPPORTED;
+}
+
+// The same without kept first keys or a gate by element.
+SANDY_API int sandy_prefill_attention_bias(const void* q, int ld_q, const void* k_cache, const void* v_cache,
+                                      long long page_stride, const int* block_table, int max_blocks,
+                                      const int* q_start, const int* kv_before, void* out, int ld_out, int n_seqs,
+                                      int max_q_len, int n_heads, int n_kv_heads, int head_dim, int page_size,
+                                      float scale, int window, float softcap, int chunk, int num_pages, const float* sink,
+                                      const float* out_gate, const float* dist_bias, int n_dist, int* status,
+                                      cudaStream_t stream) {
+    const SandyAttentionRules rules = {window, 0, softcap, chunk, sink, out_gate, dist_bias, n_dist, nullptr, 0, 0};
+    return sandy_prefill_attention_rules(q, ld_q, k_cache, v_cache, page_stride, block_table, max_blocks, q_start, kv_before, out,
+                                         ld_out, n_seqs, max_q_len, n_heads, n_kv_heads, head_dim, page_size, scale, &rules,
+                                         num_pages, status, stream);
 }
 
 // The same without a bias by distance.

@@ -53,12 +53,16 @@
 // a score s becomes softcap * tanh(s / softcap) before the softmax.  Softmax statistics and the accumulator are float; P is rounded
 // to bfloat16 for the product (the row sum is taken before rounding).
 //
+// With kept first keys behind a window (keep_first) the tiles of those keys come first and the tiles between them and the
+// window are left out; a gate by element is multiplied in when the output leaves its registers.
+//
 // Every wait on an mbarrier is bounded; a wait that runs out raises bit 8 of the status word
 // and the block runs to its end without waiting again (its output is then not valid).
 #include <cstring>
 #include <utility>
 #include <vector>
 
+#include "attention_rules.h"
 #include "tcgen05.cuh"
 
 namespace {
@@ -166,6 +170,7 @@ prefill_attention_tc_kernel(const __grid_constant__ CUtensorMap map_k, const __g
                             const int* __restrict__ kv_before, bf16* __restrict__ out, int ld_out, int n_heads,
                             int n_kv_heads, int page_size, float scale, int window, float softcap, int chunk,
                             int num_pages, int use_tma, const float* __restrict__ sink, const float* __restrict__ out_gate,
+                            int keep_first, const bf16* __restrict__ elem_gate, int ld_elem_gate, int gate_dim,
                             int* __restrict__ status) {
     extern __shared__ uint8_t smem_raw[];
     __shared__ int s_table[TABLE_SMEM];
@@ -192,8 +197,11 @@ prefill_attention_tc_kernel(const __grid_constant__ CUtensorMap map_k, const __g
     const int pos_last = pos_first + rows_valid - 1;
     int key_lo = window > 0 ? max(0, pos_first + 1 - window) : 0;
     if (chunk > 0) key_lo = max(key_lo, pos_first - pos_first % chunk);      // the first row's chunk starts first
-    const int kt_begin = key_lo / BN, kt_end = pos_last / BN;
-    const int n_it = kt_end - kt_begin + 1;
+    const int kt_window = key_lo / BN, kt_end = pos_last / BN;
+    // kept first keys: their tiles, as far as the window does not hold them anyway, come in front of the window's
+    const int kept_tiles = window > 0 ? min((keep_first + BN - 1) / BN, kt_window) : 0;
+    const int n_it = kept_tiles + kt_end - kt_window + 1;
+    auto tile_at = [&](int t) { return t < kept_tiles ? t : t - kept_tiles + kt_window; };
     const int kvh = h / (n_heads / n_kv_heads);
     const int* table = block_table + (size_t)s * max_blocks;
     const int tid = threadIdx.x, warp = tid >> 5;
@@ -229,7 +237,7 @@ prefill_attention_tc_kernel(const __grid_constant__ CUtensorMap map_k, const __g
     const bool runs_known = table_staged && n_it <= RUNS_SMEM && use_tma;
     if (runs_known) {
         for (int t = tid; t < n_it; t += THREADS) {
-            const int kt = kt_begin + t;
+            const int kt = tile_at(t);
             const int b0 = kt * pages_per_tile;
             int first = -1;
             if (kt * BN + BN - 1 <= pos_last && b0 + pages_per_tile <= max_blocks) {
@@ -269,7 +277,7 @@ prefill_attention_tc_kernel(const __grid_constant__ CUtensorMap map_k, const __g
             const int page = b < max_blocks ? (table_staged ? s_table[b] : table[b]) : -1;
             if (page < 0 || page >= num_pages) {
                 // a key with no page behind it; inside the visible range this is a fault
-                if (j >= key_lo && status && cc == 0) atomicOr(status, 16);
+                if ((j >= key_lo || j < keep_first) && status && cc == 0) atomicOr(status, 16);
                 ok = false;
             } else {
                 off = (size_t)page * page_stride + ((size_t)kvh * page_size + (j & page_mask)) * HD + cc * 8;
@@ -296,7 +304,7 @@ prefill_attention_tc_kernel(const __grid_constant__ CUtensorMap map_k, const __g
         } else if (softmax) {
             if (first < 0) {
 #pragma unroll
-                for (int i = 0; i < 4; i++) load_piece(k_cache, k_tile(t), kt_begin + t, i);
+                for (int i = 0; i < 4; i++) load_piece(k_cache, k_tile(t), tile_at(t), i);
             }
             cp_async_commit();
         }
@@ -313,7 +321,7 @@ prefill_attention_tc_kernel(const __grid_constant__ CUtensorMap map_k, const __g
         } else if (softmax) {
             if (first < 0) {
 #pragma unroll
-                for (int i = 0; i < 4; i++) load_piece(v_cache, v_tile(t), kt_begin + t, i);
+                for (int i = 0; i < 4; i++) load_piece(v_cache, v_tile(t), tile_at(t), i);
             }
             cp_async_commit();
         }
@@ -397,7 +405,7 @@ prefill_attention_tc_kernel(const __grid_constant__ CUtensorMap map_k, const __g
         const float over_cap = CAPPED ? scale / softcap : 0.0f, cap_over = CAPPED ? softcap / scale : 0.0f;
 
         for (int it = 0; it < n_it; it++) {
-            const int kt = kt_begin + it;
+            const int kt = tile_at(it);
             wait_for(&bar_s, it & 1);       // S of this tile is complete
             tc_fence_after();
             if (it + K_TILES < n_it) load_k(it + K_TILES); else cp_async_commit();      // into the tile S just left
@@ -422,8 +430,8 @@ prefill_attention_tc_kernel(const __grid_constant__ CUtensorMap map_k, const __g
             if (!whole) {
 #pragma unroll
                 for (int e = 0; e < 32; e++) {
-                    if (j0 + e > pos || j0 + e < lo) sa[e] = __float_as_uint(-INFINITY);
-                    if (j0 + 32 + e > pos || j0 + 32 + e < lo) sb[e] = __float_as_uint(-INFINITY);
+                    if (j0 + e > pos || (j0 + e < lo && j0 + e >= keep_first)) sa[e] = __float_as_uint(-INFINITY);
+                    if (j0 + 32 + e > pos || (j0 + 32 + e < lo && j0 + 32 + e >= keep_first)) sb[e] = __float_as_uint(-INFINITY);
                 }
             }
             float mx[4] = {-INFINITY, -INFINITY, -INFINITY, -INFINITY};
@@ -508,6 +516,12 @@ prefill_attention_tc_kernel(const __grid_constant__ CUtensorMap map_k, const __g
             float inv = l > 0.0f ? 1.0f / l : 0.0f;
             if (out_gate) inv *= out_gate[(size_t)(qs + t0 + row) * n_heads + h];
             bf16* dst = out + (size_t)(qs + t0 + row) * ld_out + h * HD + half * 32;
+            if (elem_gate) {
+#pragma unroll
+                for (int e = 0; e < 32; e++)
+                    r[e] = __float_as_uint(__uint_as_float(r[e]) *
+                                           elem_gate_of(elem_gate, ld_elem_gate, gate_dim, qs + t0 + row, h, half * 32 + e));
+            }
 #pragma unroll
             for (int g = 0; g < 4; g++) {
                 uint4 pk;
@@ -572,13 +586,19 @@ bool get_page_map(const void* cache, long long page_stride, int num_pages, int n
 // Arguments as sandy_prefill_attention (attention_prefill.cu).  Heads of 64 only; out and q rows
 // must be 16-byte aligned.  SANDY_ERR_UNSUPPORTED for everything else: the caller then takes the
 // mma.sync kernel.
-SANDY_API int sandy_prefill_attention_tc_cap(const void* q, int ld_q, const void* k_cache, const void* v_cache,
+SANDY_API int sandy_prefill_attention_tc_rules(const void* q, int ld_q, const void* k_cache, const void* v_cache,
                                          long long page_stride, const int* block_table, int max_blocks,
                                          const int* q_start, const int* kv_before, void* out, int ld_out, int n_seqs,
                                          int max_q_len, int n_heads, int n_kv_heads, int head_dim, int page_size,
-                                         float scale, int window, float softcap, int chunk, int num_pages,
-                                         const float* sink, const float* out_gate, int* status, cudaStream_t stream) {
+                                         float scale, const SandyAttentionRules* rules, int num_pages, int* status,
+                                         cudaStream_t stream) {
     if (n_seqs == 0 || max_q_len == 0) return SANDY_OK;
+    if (!rules) return SANDY_ERR_ARGUMENT;
+    const int window = rules->window, chunk = rules->chunk;
+    const float softcap = rules->softcap;
+    if (rules->dist_bias) return SANDY_ERR_UNSUPPORTED;              // no form for a bias by distance
+    if (rules->keep_first < 0 || (rules->keep_first > 0 && chunk > 0) || (rules->elem_gate && rules->gate_dim < 1))
+        return SANDY_ERR_UNSUPPORTED;
     if (!q || !k_cache || !v_cache || !block_table || !q_start || !kv_before || !out) return SANDY_ERR_ARGUMENT;
     if (head_dim != HD) return SANDY_ERR_UNSUPPORTED;
     if (n_kv_heads <= 0 || n_heads % n_kv_heads != 0 || page_size <= 0 || window < 0) return SANDY_ERR_UNSUPPORTED;
@@ -612,7 +632,21 @@ SANDY_API int sandy_prefill_attention_tc_cap(const void* q, int ld_q, const void
     return sandy_launch(softcap > 0.0f ? prefill_attention_tc_kernel<true> : prefill_attention_tc_kernel<false>, grid, dim3(THREADS), SMEM_BYTES, stream, mk, mv, (const bf16*)q, ld_q,
                         (const bf16*)k_cache, (const bf16*)v_cache, page_stride, block_table, max_blocks, q_start,
                         kv_before, (bf16*)out, ld_out, n_heads, n_kv_heads, page_size, scale, window, softcap, chunk, num_pages,
-                        use_tma, sink, out_gate, status);
+                        use_tma, rules->sink, rules->out_gate, rules->keep_first, (const bf16*)rules->elem_gate,
+                        rules->ld_elem_gate, rules->gate_dim, status);
+}
+
+// The same without kept first keys or a gate by element.
+SANDY_API int sandy_prefill_attention_tc_cap(const void* q, int ld_q, const void* k_cache, const void* v_cache,
+                                         long long page_stride, const int* block_table, int max_blocks,
+                                         const int* q_start, const int* kv_before, void* out, int ld_out, int n_seqs,
+                                         int max_q_len, int n_heads, int n_kv_heads, int head_dim, int page_size,
+                                         float scale, int window, float softcap, int chunk, int num_pages,
+                                         const float* sink, const float* out_gate, int* status, cudaStream_t stream) {
+    const SandyAttentionRules rules = {window, 0, softcap, chunk, sink, out_gate, nullptr, 0, nullptr, 0, 0};
+    return sandy_prefill_attention_tc_rules(q, ld_q, k_cache, v_cache, page_stride, block_table, max_blocks, q_start, kv_before,
+                                            out, ld_out, n_seqs, max_q_len, n_heads, n_kv_heads, head_dim, page_size, scale,
+                                            &rules, num_pages, status, stream);
 }
 
 // The same without capped scores or chunks.

@@ -3,7 +3,7 @@
 //   1. optional RMS norm of the WHOLE query row and of the whole key row (all heads at once, one gain per
 //      element; eps inside the root), in 32-bit;
 //   2. optional rotary position encoding of queries and keys on the first `rot_dims` entries of every head
-//      ("rotate half": entry i pairs with entry i + rot_dims / 2; the pair (u, v) at position p becomes
+//      ("rotate half": entry i pairs with entry i + rot_dims / 2; or interleaved: 2i with 2i + 1; the pair (u, v) at position p becomes
 //      (u cos a - v sin a, v cos a + u sin a), a = p * freq[i]), positions and angles in 32-bit; the
 //      frequencies come from the caller, who has applied whatever rescaling the model wants;
 //   3. keys and values written into the request's pages, queries into a dense matrix, each head padded
@@ -32,7 +32,8 @@ attention_prepare_kernel(const T* __restrict__ proj, int ld, int q_off, int k_of
                          T* __restrict__ v_cache, long long page_stride, int page_size, int num_pages, int write_cache,
                          T* __restrict__ q_out, int ld_q, const float* __restrict__ gate_in, int ld_gate,
                          float* __restrict__ gate_out, float gate_scale, const float* __restrict__ q_head_scale,
-                         float v_unit_eps, int per_head_norm, float q_pos_coef, int q_pos_every, int* __restrict__ status) {
+                         float v_unit_eps, int per_head_norm, float q_pos_coef, int q_pos_every, int interleaved,
+                         int* __restrict__ status) {
     __shared__ float scratch[32];
     extern __shared__ float cs[];                    // cos [rot_dims / 2], sin [rot_dims / 2], then 1 / rms of each value head,
     float* v_inv = cs + rot_dims;                    // then (per_head_norm) 1 / rms of each query head and each key head
@@ -112,6 +113,10 @@ attention_prepare_kernel(const T* __restrict__ proj, int ld, int q_off, int k_of
         const int base = off + head * qk_dim;
         auto normed = [&](int j) { return to_f32(row[base + j]) * inv * (gain ? gain[head * qk_dim + j] : 1.0f); };
         if (!freq || i >= rot_dims) return normed(i);
+        if (interleaved) {
+            const float c = cs[i >> 1], s = cs[half + (i >> 1)];
+            return (i & 1) ? normed(i) * c + normed(i - 1) * s : normed(i) * c - normed(i + 1) * s;
+        }
         if (i < half) return normed(i) * cs[i] - normed(i + half) * cs[half + i];
         return normed(i) * cs[i - half] + normed(i - half) * cs[i];
     };
@@ -147,14 +152,16 @@ attention_prepare_kernel(const T* __restrict__ proj, int ld, int q_off, int k_of
 // per_head_norm != 0: every query head and every key head is divided by its own root mean square over qk_dim (eps inside
 // the root; the gains, [heads * qk_dim], may then be null) instead of the norm over the whole row.  q_pos_every > 0: the
 // query at position p is multiplied by 1 + q_pos_coef * ln(floor((p + 1) / q_pos_every) + 1).
-SANDY_API int sandy_attention_prepare_pos(const void* proj, int ld, int q_off, int k_off, int v_off, int n_tokens, int n_heads,
+// interleaved != 0: the rotation pairs entries 2i and 2i + 1 instead of i and i + rot_dims / 2.
+SANDY_API int sandy_attention_prepare_rot(const void* proj, int ld, int q_off, int k_off, int v_off, int n_tokens, int n_heads,
                                       int n_kv_heads, int qk_dim, int v_dim, int pad_dim, const float* q_gain,
                                       const float* k_gain, float eps, const float* freq, int rot_dims, const int* positions,
                                       const int* token_seq, const int* block_table, int max_blocks, void* k_cache,
                                       void* v_cache, long long page_stride, int page_size, int num_pages, int write_cache,
                                       void* q_out, int ld_q, const float* gate_in, int ld_gate, float* gate_out,
                                       float gate_scale, const float* q_head_scale, float v_unit_eps, int per_head_norm,
-                                      float q_pos_coef, int q_pos_every, int dtype, int* status, cudaStream_t stream) {
+                                      float q_pos_coef, int q_pos_every, int interleaved, int dtype, int* status,
+                                      cudaStream_t stream) {
     if (n_tokens == 0) return SANDY_OK;
     if (!proj || !positions || !token_seq || !q_out || (write_cache && (!block_table || !k_cache || !v_cache)))
         return SANDY_ERR_ARGUMENT;
@@ -167,14 +174,30 @@ SANDY_API int sandy_attention_prepare_pos(const void* proj, int ld, int q_off, i
                             ld, q_off, k_off, v_off, n_heads, n_kv_heads, qk_dim, v_dim, pad_dim, q_gain, k_gain, eps, freq,
                             rot_dims, positions, token_seq, block_table, max_blocks, (float*)k_cache, (float*)v_cache,
                             page_stride, page_size, num_pages, write_cache, (float*)q_out, ld_q, gate_in, ld_gate, gate_out,
-                            gate_scale, q_head_scale, v_unit_eps, per_head_norm, q_pos_coef, q_pos_every, status);
+                            gate_scale, q_head_scale, v_unit_eps, per_head_norm, q_pos_coef, q_pos_every, interleaved, status);
     if (dtype == SANDY_BF16)
         return sandy_launch(attention_prepare_kernel<bf16>, dim3(n_tokens), dim3(THREADS), smem, stream, (const bf16*)proj,
                             ld, q_off, k_off, v_off, n_heads, n_kv_heads, qk_dim, v_dim, pad_dim, q_gain, k_gain, eps, freq,
                             rot_dims, positions, token_seq, block_table, max_blocks, (bf16*)k_cache, (bf16*)v_cache,
                             page_stride, page_size, num_pages, write_cache, (bf16*)q_out, ld_q, gate_in, ld_gate, gate_out,
-                            gate_scale, q_head_scale, v_unit_eps, per_head_norm, q_pos_coef, q_pos_every, status);
+                            gate_scale, q_head_scale, v_unit_eps, per_head_norm, q_pos_coef, q_pos_every, interleaved, status);
     return SANDY_ERR_UNSUPPORTED;
+}
+
+// The same with the rotation's pairs half a rotated part apart.
+SANDY_API int sandy_attention_prepare_pos(const void* proj, int ld, int q_off, int k_off, int v_off, int n_tokens, int n_heads,
+                                      int n_kv_heads, int qk_dim, int v_dim, int pad_dim, const float* q_gain,
+                                      const float* k_gain, float eps, const float* freq, int rot_dims, const int* positions,
+                                      const int* token_seq, const int* block_table, int max_blocks, void* k_cache,
+                                      void* v_cache, long long page_stride, int page_size, int num_pages, int write_cache,
+                                      void* q_out, int ld_q, const float* gate_in, int ld_gate, float* gate_out,
+                                      float gate_scale, const float* q_head_scale, float v_unit_eps, int per_head_norm,
+                                      float q_pos_coef, int q_pos_every, int dtype, int* status, cudaStream_t stream) {
+    return sandy_attention_prepare_rot(proj, ld, q_off, k_off, v_off, n_tokens, n_heads, n_kv_heads, qk_dim, v_dim, pad_dim, q_gain,
+                                       k_gain, eps, freq, rot_dims, positions, token_seq, block_table, max_blocks, k_cache, v_cache,
+                                       page_stride, page_size, num_pages, write_cache, q_out, ld_q, gate_in, ld_gate, gate_out,
+                                       gate_scale, q_head_scale, v_unit_eps, per_head_norm, q_pos_coef, q_pos_every, 0, dtype, status,
+                                       stream);
 }
 
 // The same with the norms over whole rows and no factor by position.

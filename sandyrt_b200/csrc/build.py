@@ -52,6 +52,7 @@ LIBRARIES: Dict[str, List[str]] = {
     "elementwise": [],
     "attention_prepare": [],
     "matrix_state": [],
+    "gated_linear": [],
     "latent_prepare": [],
     "grouped_gemm": [],
     "grouped_gemm_tc": [],

@@ -53,6 +53,28 @@ __device__ __forceinline__ float warp_max(float v) {
     return v;
 }
 
+// The keys a query at position pos sees, numbered 0 .. n - 1 in the order of their positions: the sequence's first `kept`
+// positions where a window has left them behind, then the run lo .. pos.
+struct VisibleKeys {
+    int lo, kept, n;
+    __device__ __forceinline__ int position(int v) const { return v < kept ? v : v - kept + lo; }
+};
+__device__ __forceinline__ VisibleKeys visible_keys(int pos, int window, int keep_first, int chunk) {
+    VisibleKeys k;
+    k.lo = window > 0 ? max(0, pos + 1 - window) : 0;
+    if (chunk > 0) k.lo = max(k.lo, pos - pos % chunk);
+    k.kept = min(keep_first, k.lo);
+    k.n = k.kept + pos + 1 - k.lo;
+    return k;
+}
+
+// sigmoid of a gate's pre-activation, for element i of head h of token t (1 where there is no gate, or behind its `dim`).
+template <typename T>
+__device__ __forceinline__ float elem_gate_of(const T* __restrict__ gate, int ld, int dim, int t, int h, int i) {
+    if (!gate || i >= dim) return 1.0f;
+    return 1.0f / (1.0f + expf(-to_f32(gate[(size_t)t * ld + h * dim + i])));
+}
+
 // Sum over a block of up to 1024 threads.  `scratch` holds 32 floats.  Every thread
 // gets the total; the order of the additions is fixed by the thread layout, so the
 // result for a row does not depend on what else runs beside it.

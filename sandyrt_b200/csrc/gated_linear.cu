@@ -1,0 +1,508 @@
+// Gated linear attention: a recurrent mixer whose per-request state is a matrix per head and whose decay is one factor
+// per key channel and token.
+//
+//   z = W2 (W1 h) + b          [H * d], a product of low rank; what W1 h gives comes in as float32 rows `low` [T, rank]
+//   la = logsigmoid(z) / tau   the decay's logarithm, never above zero
+//   S_t = diag(exp(la_t)) S_(t-1) + k_t v_t^T,   o_t = S_t^T (q_t * q_scale)         S [d, e] per head
+//
+// Everything here is float32 arithmetic whatever the engine's compute type; q, k and v are read in the projection's type.
+// The state lives in the request's slot, transposed: [H][e][d], so that a column's rows are consecutive.  The columns of S
+// never meet, so every kernel spreads the work over (request, head, block of SANDY_MATRIX_STATE_COLS columns).
+//
+// Token by token (`sandy_gla_scan`): decode steps and short portions.  A warp owns four columns, a lane the rows lane,
+// lane + 32, ...; the decays of the staged tokens are formed by the block itself (rank multiplications a channel), so a
+// decode step is one launch.
+//
+// A chunk of 32 tokens at a time, in two launches.  With A_t the running sum of la inside the chunk and S0 the state
+// before it,
+//   o_t = (q_t exp(A_t))^T S0 + sum_{j<=t} P(t, j) v_j,   P(t, j) = sum_i q_t[i] k_j[i] exp(A_t[i] - A_j[i])
+//   S   = diag(exp(A_31)) S0 + sum_j (k_j exp(A_31 - A_j)) v_j^T
+// Splitting exp(A_t - A_j) into exp(A_t) exp(-A_j) would overflow where a channel fades fast, so the chunk is cut into
+// four parts of 8 tokens and only exponents that are never positive are formed.  With L the running sum inside a part and
+// D_r a part's whole sum: inside a part exp(L_t - L_j) is formed pair by pair; between parts r < s
+// exp(L_t) * exp(D_(r+1) + .. + D_(s-1)) * exp(D_r - L_j).
+//   sandy_gla_chunk_prepare   one block a (chunk, head, request), all chunks side by side: P, q exp(A_t), k exp(A_31 - A_j)
+//                             and exp(A_31), in float32
+//   sandy_gla_chunk_scan      one block a (request, head, 16 columns) walks the chunks with S in shared memory; nothing
+//                             that does not need the state is left in it.  The next chunk's rows come by cp.async while
+//                             this one is computed.
+#include "common.cuh"
+#include "matrix_state.h"
+
+namespace {
+
+constexpr int WARPS = 4;
+constexpr int CPW = 4;                                   // columns per warp
+constexpr int COLS = SANDY_MATRIX_STATE_COLS;            // columns per block
+static_assert(COLS == WARPS * CPW, "a block's columns are its warps' columns");
+constexpr int THREADS = WARPS * 32;
+constexpr int STAGE = 8;                                 // tokens staged at a time, token by token
+
+__device__ __forceinline__ float log_sigmoid_f(float z) { return fminf(z, 0.0f) - log1pf(expf(-fabsf(z))); }
+
+// ---- token by token ------------------------------------------------------------------------------------------
+// Shared memory per staged token: q [d], k [d], decay [d], v [COLS].
+template <typename T, int R>
+__global__ void __launch_bounds__(THREADS)
+gla_scan_kernel(const T* __restrict__ proj, int ld, int q_off, int k_off, int v_off, const float* __restrict__ low, int ld_low,
+                int rank, const float* __restrict__ w2t, const float* __restrict__ bias, float inv_tau, float q_scale,
+                float* __restrict__ state, long long state_stride, const int* __restrict__ q_start,
+                const int* __restrict__ seq_slots, float* __restrict__ out, int ld_out, int n_heads, int d, int e, int long_from) {
+    extern __shared__ float stage[];
+    const int s = blockIdx.x, h = blockIdx.y, col0 = blockIdx.z * COLS;
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    const int per = 3 * d + COLS;
+    const int t0 = q_start[s], t1 = q_start[s + 1];
+    if (long_from > 0 && t1 - t0 >= long_from) {
+        pdl_wait();                                      // a kernel ends only after the one before it has
+        return;
+    }
+    float* S = state + (long long)seq_slots[s] * state_stride + (long long)h * e * d;    // [e][d]
+    pdl_wait();
+    float st[R][CPW];
+#pragma unroll
+    for (int c = 0; c < CPW; c++) {
+        const int col = col0 + warp * CPW + c;
+#pragma unroll
+        for (int r = 0; r < R; r++) {
+            const int i = lane + 32 * r;
+            st[r][c] = (col < e && i < d) ? S[(size_t)col * d + i] : 0.0f;
+        }
+    }
+    for (int tc = t0; tc < t1; tc += STAGE) {
+        const int n_tok = min(STAGE, t1 - tc);
+        __syncthreads();
+        for (int f = threadIdx.x; f < n_tok * d; f += THREADS) {
+            const int tok = f / d, i = f % d, ch = h * d + i;
+            const T* row = proj + (size_t)(tc + tok) * ld;
+            float* dst = stage + tok * per;
+            dst[i] = to_f32(row[q_off + ch]) * q_scale;
+            dst[d + i] = to_f32(row[k_off + ch]);
+            float z = bias[ch];
+            const float* lo = low + (size_t)(tc + tok) * ld_low;
+            for (int r = 0; r < rank; r++) z = fmaf(w2t[(size_t)r * n_heads * d + ch], lo[r], z);
+            dst[2 * d + i] = expf(log_sigmoid_f(z) * inv_tau);
+        }
+        for (int f = threadIdx.x; f < n_tok * COLS; f += THREADS) {
+            const int tok = f / COLS, c = f % COLS;
+            stage[tok * per + 3 * d + c] = col0 + c < e ? to_f32(proj[(size_t)(tc + tok) * ld + v_off + h * e + col0 + c]) : 0.0f;
+        }
+        __syncthreads();
+        for (int tok = 0; tok < n_tok; tok++) {
+            const float* in = stage + tok * per;
+            float v[CPW], red[CPW];
+#pragma unroll
+            for (int c = 0; c < CPW; c++) {
+                v[c] = in[3 * d + warp * CPW + c];
+                red[c] = 0.0f;
+            }
+#pragma unroll
+            for (int r = 0; r < R; r++) {
+                const int i = lane + 32 * r;
+                if (i < d) {
+                    const float q = in[i], k = in[d + i], a = in[2 * d + i];
+#pragma unroll
+                    for (int c = 0; c < CPW; c++) {
+                        st[r][c] = fmaf(k, v[c], a * st[r][c]);
+                        red[c] = fmaf(st[r][c], q, red[c]);
+                    }
+                }
+            }
+#pragma unroll
+            for (int o = 16; o > 0; o >>= 1)
+#pragma unroll
+                for (int c = 0; c < CPW; c++) red[c] += __shfl_xor_sync(0xffffffffu, red[c], o);
+            float mine = red[0];
+#pragma unroll
+            for (int c = 1; c < CPW; c++)
+                if (lane == c) mine = red[c];
+            const int col = col0 + warp * CPW + lane;
+            if (lane < CPW && col < e) out[(size_t)(tc + tok) * ld_out + h * e + col] = mine;
+        }
+    }
+    pdl_launch_dependents();
+    if (t0 < t1) {
+#pragma unroll
+        for (int c = 0; c < CPW; c++) {
+            const int col = col0 + warp * CPW + c;
+#pragma unroll
+            for (int r = 0; r < R; r++) {
+                const int i = lane + 32 * r;
+                if (col < e && i < d) S[(size_t)col * d + i] = st[r][c];
+            }
+        }
+    }
+}
+
+// ---- chunks: what does not need the state --------------------------------------------------------------------
+constexpr int CC = 32;                 // tokens per chunk
+constexpr int CT = 256;                // threads
+constexpr int PART = 8;                // tokens per part
+constexpr int PARTS = CC / PART;
+static_assert(CT == PARTS * PART * PART, "inside the parts a thread a pair");
+
+// Place of chunk c of request s among all chunks of the step (a request brings ceil(n / CC) of them).
+__device__ __forceinline__ int chunk_slot(int t0, int s, int c) { return t0 / CC + s + c; }
+
+__device__ __forceinline__ float dot4(const float* __restrict__ x, const float* __restrict__ y, int n) {
+    float a = 0.0f, b = 0.0f;
+    for (int i = 0; i < n; i += 4) {
+        const float4 u = *reinterpret_cast<const float4*>(x + i), v = *reinterpret_cast<const float4*>(y + i);
+        a = fmaf(u.x, v.x, a);
+        b = fmaf(u.y, v.y, b);
+        a = fmaf(u.z, v.z, a);
+        b = fmaf(u.w, v.w, b);
+    }
+    return a + b;
+}
+
+// qs, ks: float32 [T, H * dp]; P: float32 [T, H * CC]; dec: float32 [slots, H * dp]; dp = d rounded up to 4, zeros behind d.
+template <typename T>
+__global__ void __launch_bounds__(CT)
+gla_chunk_prepare_kernel(const T* __restrict__ proj, int ld, int q_off, int k_off, const float* __restrict__ low, int ld_low,
+                         int rank, const float* __restrict__ w2t, const float* __restrict__ bias, float inv_tau, float q_scale,
+                         const int* __restrict__ q_start, float* __restrict__ qs, float* __restrict__ ks, float* __restrict__ P,
+                         float* __restrict__ dec, int n_heads, int d, int long_from) {
+    extern __shared__ __align__(16) float smem[];
+    const int c = blockIdx.x, h = blockIdx.y, s = blockIdx.z, tid = threadIdx.x;
+    const int t0 = q_start[s], n = q_start[s + 1] - t0;
+    pdl_wait();
+    if (n < long_from || c * CC >= n) return;
+    const int tc = t0 + c * CC, n_tok = min(CC, n - c * CC);
+    const int dp = (d + 3) / 4 * 4, lds = dp + 4;
+    float* sq = smem;                     // [CC][lds]
+    float* sk = sq + CC * lds;            // [CC][lds]
+    float* sl = sk + CC * lds;            // [CC][lds]: L
+    float* sp = sl + CC * lds;            // [CC][CC]
+    float* slow = sp + CC * CC;           // [CC][rank]
+    for (int x = tid; x < CC * dp; x += CT) {
+        const int t = x / dp, i = x % dp;
+        const bool live = t < n_tok && i < d;
+        const T* row = proj + (size_t)(tc + (live ? t : 0)) * ld;
+        sq[t * lds + i] = live ? to_f32(row[q_off + h * d + i]) * q_scale : 0.0f;
+        sk[t * lds + i] = live ? to_f32(row[k_off + h * d + i]) : 0.0f;
+    }
+    for (int x = tid; x < CC * rank; x += CT) {
+        const int t = x / rank, r = x % rank;
+        slow[x] = t < n_tok ? low[(size_t)(tc + t) * ld_low + r] : 0.0f;
+    }
+    for (int x = tid; x < CC * CC; x += CT) sp[x] = 0.0f;
+    __syncthreads();
+    // the decays' logarithms and their running sums inside a part: a thread a (channel, part)
+    for (int x = tid; x < PARTS * dp; x += CT) {
+        const int part = x / dp, i = x % dp;
+        float z[PART];
+        if (i < d) {
+            const float b = bias[h * d + i];
+#pragma unroll
+            for (int t = 0; t < PART; t++) z[t] = b;
+            for (int r = 0; r < rank; r++) {
+                const float w = w2t[(size_t)r * n_heads * d + h * d + i];
+#pragma unroll
+                for (int t = 0; t < PART; t++) z[t] = fmaf(w, slow[(part * PART + t) * rank + r], z[t]);
+            }
+        }
+        float run = 0.0f;
+#pragma unroll
+        for (int t = 0; t < PART; t++) {
+            if (i < d && part * PART + t < n_tok) run += log_sigmoid_f(z[t]) * inv_tau;
+            sl[(part * PART + t) * lds + i] = run;
+        }
+    }
+    __syncthreads();
+    // pairs inside a part, a thread a pair
+    {
+        const int part = tid / (PART * PART), tt = part * PART + (tid / PART) % PART, jj = part * PART + tid % PART;
+        if (jj <= tt) {
+            const float *q = sq + tt * lds, *k = sk + jj * lds, *lt = sl + tt * lds, *lj = sl + jj * lds;
+            float a = 0.0f;
+            if (jj == tt) a = dot4(q, k, dp);
+            else
+                for (int i = 0; i < dp; i += 4) {
+                    const float4 qv = *reinterpret_cast<const float4*>(q + i), kv = *reinterpret_cast<const float4*>(k + i);
+                    const float4 u = *reinterpret_cast<const float4*>(lt + i), v = *reinterpret_cast<const float4*>(lj + i);
+                    a = fmaf(qv.x * kv.x, expf(u.x - v.x), a);
+                    a = fmaf(qv.y * kv.y, expf(u.y - v.y), a);
+                    a = fmaf(qv.z * kv.z, expf(u.z - v.z), a);
+                    a = fmaf(qv.w * kv.w, expf(u.w - v.w), a);
+                }
+            sp[tt * CC + jj] = a;
+        }
+    }
+    __syncthreads();
+    for (int x = tid; x < CC * dp; x += CT) {             // q exp(L), k exp(D - L)
+        const int t = x / dp, i = x % dp, last = (t / PART) * PART + PART - 1;
+        const float l = sl[t * lds + i];
+        sq[t * lds + i] *= expf(l);
+        sk[t * lds + i] *= expf(sl[last * lds + i] - l);
+    }
+    __syncthreads();
+    // pairs between parts: the keys of earlier parts fade on by one part's sum a round
+    for (int p = 1; p < PARTS; p++) {
+        if (p > 1) {
+            for (int x = tid; x < (p - 1) * PART * dp; x += CT) {
+                const int t = x / dp, i = x % dp;
+                sk[t * lds + i] *= expf(sl[(p * PART - 1) * lds + i]);
+            }
+            __syncthreads();
+        }
+        const int keys = p * PART;
+        if (tid < PART * keys) {
+            const int t = p * PART + tid / keys, j = tid % keys;
+            sp[t * CC + j] = dot4(sq + t * lds, sk + j * lds, dp);
+        }
+        __syncthreads();
+    }
+    // out: queries as seen from the chunk's start, keys as seen from its end, the whole chunk's fading, P
+    const int ldw = n_heads * dp;
+    for (int x = tid; x < n_tok * dp; x += CT) {
+        const int t = x / dp, i = x % dp, part = t / PART;
+        float before = 0.0f;
+        for (int p = 0; p < part; p++) before += sl[(p * PART + PART - 1) * lds + i];
+        qs[(size_t)(tc + t) * ldw + h * dp + i] = sq[t * lds + i] * expf(before);
+        const float k = sk[t * lds + i];
+        ks[(size_t)(tc + t) * ldw + h * dp + i] = part < PARTS - 1 ? k * expf(sl[(CC - 1) * lds + i]) : k;
+    }
+    for (int i = tid; i < dp; i += CT) {
+        float all = 0.0f;
+#pragma unroll
+        for (int p = 0; p < PARTS; p++) all += sl[(p * PART + PART - 1) * lds + i];
+        dec[(size_t)chunk_slot(t0, s, c) * ldw + h * dp + i] = expf(all);
+    }
+    for (int x = tid; x < n_tok * CC; x += CT) P[((size_t)(tc + x / CC) * n_heads + h) * CC + x % CC] = sp[x];
+    pdl_launch_dependents();
+}
+
+// ---- chunks: the recurrence ------------------------------------------------------------------------------------
+__device__ __forceinline__ void cp16(void* smem, const void* gmem, bool valid) {
+    const unsigned dst = (unsigned)__cvta_generic_to_shared(smem);
+    const int bytes = valid ? 16 : 0;
+    asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(dst), "l"(gmem), "r"(bytes) : "memory");
+}
+
+__host__ __device__ constexpr int scan_buffer_floats(int dp) { return 2 * CC * dp + CC * CC + dp; }      // q, k, P, dec
+
+// MAXR: rows of the state a thread owns (d <= 32 * MAXR).
+template <typename T, int MAXR>
+__global__ void __launch_bounds__(CT)
+gla_chunk_scan_kernel(const T* __restrict__ proj, int ld, int v_off, const float* __restrict__ qs, const float* __restrict__ ks,
+                      const float* __restrict__ P, const float* __restrict__ dec, float* __restrict__ state, long long state_stride,
+                      const int* __restrict__ q_start, const int* __restrict__ seq_slots, float* __restrict__ out, int ld_out,
+                      int n_heads, int d, int e, int long_from) {
+    extern __shared__ __align__(16) float smem[];
+    const int s = blockIdx.x, h = blockIdx.y, col0 = blockIdx.z * COLS, tid = threadIdx.x;
+    const int t0 = q_start[s], t1 = q_start[s + 1];
+    pdl_wait();
+    if (t1 - t0 < long_from) return;
+    const int dp = (d + 3) / 4 * 4, ldw = n_heads * dp, buf_floats = scan_buffer_floats(dp);
+    float* buf = smem;                              // two of (q [CC][dp], k [CC][dp], P [CC][CC], dec [dp])
+    float* sv = buf + 2 * buf_floats;               // [CC][COLS]
+    float* S0 = sv + CC * COLS;                     // [dp][COLS]
+    float* S = state + (long long)seq_slots[s] * state_stride + (long long)h * e * d;
+    for (int x = tid; x < dp * COLS; x += CT) {
+        const int c = x / dp, i = x % dp;            // consecutive threads read consecutive rows of a column
+        S0[i * COLS + c] = (i < d && col0 + c < e) ? S[(size_t)(col0 + c) * d + i] : 0.0f;
+    }
+    float pre_v[CC * COLS / CT];
+    auto fetch = [&](int tc, int b) {                // chunk at token tc into buffer b; nothing behind the last token
+        float* dst = buf + b * buf_floats;
+        const int n_tok = t1 - tc, pieces = dp / 4;
+        for (int x = tid; x < CC * pieces; x += CT) {
+            const int t = x / pieces, i = (x % pieces) * 4;
+            const bool live = t < n_tok;
+            const size_t at = (size_t)(live ? tc + t : t0) * ldw + h * dp + i;
+            cp16(dst + t * dp + i, qs + at, live);
+            cp16(dst + CC * dp + t * dp + i, ks + at, live);
+        }
+        for (int x = tid; x < CC * CC / 4; x += CT) {
+            const int t = x / (CC / 4), j = (x % (CC / 4)) * 4;
+            const bool live = t < n_tok;
+            cp16(dst + 2 * CC * dp + t * CC + j, P + ((size_t)(live ? tc + t : t0) * n_heads + h) * CC + j, live);
+        }
+        for (int x = tid; x < pieces; x += CT)
+            cp16(dst + 2 * CC * dp + CC * CC + x * 4, dec + (size_t)chunk_slot(t0, s, n_tok > 0 ? (tc - t0) / CC : 0) * ldw + h * dp + x * 4, true);
+        asm volatile("cp.async.commit_group;" ::: "memory");
+#pragma unroll
+        for (int u = 0; u < CC * COLS / CT; u++) {
+            const int x = tid + u * CT, t = x / COLS, c = x % COLS;
+            pre_v[u] = (t < n_tok && col0 + c < e) ? to_f32(proj[(size_t)(tc + t) * ld + v_off + h * e + col0 + c]) : 0.0f;
+        }
+    };
+    const int ot = tid / 8, oc = (tid % 8) * 2;      // this thread's token (and first state row) and two columns
+    fetch(t0, 0);
+    for (int tc = t0, b = 0; tc < t1; tc += CC, b ^= 1) {
+        const int n_tok = min(CC, t1 - tc);
+        __syncthreads();                             // everyone is done with sv and the other buffer
+#pragma unroll
+        for (int u = 0; u < CC * COLS / CT; u++) sv[tid + u * CT] = pre_v[u];
+        const bool more = tc + CC < t1;
+        if (more) fetch(tc + CC, b ^ 1);
+        if (more) asm volatile("cp.async.wait_group 1;" ::: "memory");
+        else asm volatile("cp.async.wait_group 0;" ::: "memory");
+        __syncthreads();
+        const float* q = buf + b * buf_floats;
+        const float* k = q + CC * dp;
+        const float* p = k + CC * dp;
+        const float* fade = p + CC * CC;
+        float o[2] = {0.0f, 0.0f};
+        {
+            const float* qrow = q + ot * dp;
+            for (int i = 0; i < dp; i += 4) {
+                const float4 x = *reinterpret_cast<const float4*>(qrow + i);
+                const float2 a0 = *reinterpret_cast<const float2*>(S0 + (i + 0) * COLS + oc), a1 = *reinterpret_cast<const float2*>(S0 + (i + 1) * COLS + oc);
+                const float2 a2 = *reinterpret_cast<const float2*>(S0 + (i + 2) * COLS + oc), a3 = *reinterpret_cast<const float2*>(S0 + (i + 3) * COLS + oc);
+                o[0] = fmaf(x.x, a0.x, o[0]); o[1] = fmaf(x.x, a0.y, o[1]);
+                o[0] = fmaf(x.y, a1.x, o[0]); o[1] = fmaf(x.y, a1.y, o[1]);
+                o[0] = fmaf(x.z, a2.x, o[0]); o[1] = fmaf(x.z, a2.y, o[1]);
+                o[0] = fmaf(x.w, a3.x, o[0]); o[1] = fmaf(x.w, a3.y, o[1]);
+            }
+            const float* prow = p + ot * CC;
+            for (int j = 0; j <= ot; j += 4) {       // P is zero behind the diagonal, v behind the last token
+                const float4 x = *reinterpret_cast<const float4*>(prow + j);
+                const float2 a0 = *reinterpret_cast<const float2*>(sv + (j + 0) * COLS + oc), a1 = *reinterpret_cast<const float2*>(sv + (j + 1) * COLS + oc);
+                const float2 a2 = *reinterpret_cast<const float2*>(sv + (j + 2) * COLS + oc), a3 = *reinterpret_cast<const float2*>(sv + (j + 3) * COLS + oc);
+                o[0] = fmaf(x.x, a0.x, o[0]); o[1] = fmaf(x.x, a0.y, o[1]);
+                o[0] = fmaf(x.y, a1.x, o[0]); o[1] = fmaf(x.y, a1.y, o[1]);
+                o[0] = fmaf(x.z, a2.x, o[0]); o[1] = fmaf(x.z, a2.y, o[1]);
+                o[0] = fmaf(x.w, a3.x, o[0]); o[1] = fmaf(x.w, a3.y, o[1]);
+            }
+            if (ot < n_tok)
+#pragma unroll
+                for (int c = 0; c < 2; c++)
+                    if (col0 + oc + c < e) out[(size_t)(tc + ot) * ld_out + h * e + col0 + oc + c] = o[c];
+        }
+        // the state after the chunk, kept in registers until everyone has read S0
+        float sn[MAXR][2];
+#pragma unroll
+        for (int r = 0; r < MAXR; r++) {
+            const int i = ot + 32 * r;
+            if (i < dp) {
+                const float2 x = *reinterpret_cast<const float2*>(S0 + i * COLS + oc);
+                const float f = fade[i];
+                sn[r][0] = f * x.x; sn[r][1] = f * x.y;
+            }
+        }
+        for (int j = 0; j < n_tok; j++) {
+            const float2 v = *reinterpret_cast<const float2*>(sv + j * COLS + oc);
+#pragma unroll
+            for (int r = 0; r < MAXR; r++) {
+                const int i = ot + 32 * r;
+                if (i < dp) {
+                    const float x = k[j * dp + i];
+                    sn[r][0] = fmaf(x, v.x, sn[r][0]); sn[r][1] = fmaf(x, v.y, sn[r][1]);
+                }
+            }
+        }
+        __syncthreads();
+#pragma unroll
+        for (int r = 0; r < MAXR; r++) {
+            const int i = ot + 32 * r;
+            if (i < dp) *reinterpret_cast<float2*>(S0 + i * COLS + oc) = make_float2(sn[r][0], sn[r][1]);
+        }
+    }
+    __syncthreads();
+    pdl_launch_dependents();
+    for (int x = tid; x < dp * COLS; x += CT) {
+        const int c = x / dp, i = x % dp;
+        if (i < d && col0 + c < e) S[(size_t)(col0 + c) * d + i] = S0[i * COLS + c];
+    }
+}
+
+size_t prepare_smem(int d, int rank) {
+    const int dp = (d + 3) / 4 * 4;
+    return (size_t)(3 * CC * (dp + 4) + CC * CC + CC * rank) * sizeof(float);
+}
+size_t scan_smem(int d) {
+    const int dp = (d + 3) / 4 * 4;
+    return (size_t)(2 * scan_buffer_floats(dp) + CC * COLS + dp * COLS) * sizeof(float);
+}
+
+constexpr int MAX_DIM = 256, MAX_RANK = 512;
+
+template <typename K>
+int allow_smem(K kernel, size_t smem, size_t& configured) {
+    if (smem <= 48 * 1024 || smem <= configured) return SANDY_OK;
+    const cudaError_t err = cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+    if (err != cudaSuccess) return (int)err;
+    configured = smem;
+    return SANDY_OK;
+}
+
+}  // namespace
+
+// proj: [T, ld] of dtype with q at q_off + h * qk_dim, k at k_off + h * qk_dim, v at v_off + h * v_dim; low: float32
+// [T, rank] with pitch ld_low; w2t: float32 [rank, n_heads * qk_dim]; bias: float32 [n_heads * qk_dim]; state: float32, a
+// request's S [n_heads][v_dim][qk_dim] at the start of its slot; out: float32 [T, n_heads * v_dim].  Requests that bring
+// `long_from` tokens or more are left to the chunked kernels (0: none are).
+SANDY_API int sandy_gla_scan(const void* proj, int ld, int dtype, int q_off, int k_off, int v_off, const float* low, int ld_low,
+                             int rank, const float* w2t, const float* bias, float inv_tau, float q_scale, float* state,
+                             long long state_stride, const int* q_start, const int* seq_slots, float* out, int ld_out, int n_seqs,
+                             int n_heads, int qk_dim, int v_dim, int long_from, cudaStream_t stream) {
+    if (n_seqs == 0) return SANDY_OK;
+    if (!proj || !low || !w2t || !bias || !state || !q_start || !seq_slots || !out) return SANDY_ERR_ARGUMENT;
+    if (qk_dim <= 0 || qk_dim > MAX_DIM || v_dim <= 0 || n_heads <= 0 || rank < 1 || n_heads > 65535) return SANDY_ERR_UNSUPPORTED;
+    const dim3 grid(n_seqs, n_heads, (v_dim + COLS - 1) / COLS);
+    const size_t smem = (size_t)STAGE * (3 * qk_dim + COLS) * sizeof(float);
+#define CASE(TT, RR)                                                                                                     \
+    if (qk_dim <= 32 * RR)                                                                                               \
+        return sandy_launch(gla_scan_kernel<TT, RR>, grid, dim3(THREADS), smem, stream, (const TT*)proj, ld, q_off,      \
+                            k_off, v_off, low, ld_low, rank, w2t, bias, inv_tau, q_scale, state, state_stride, q_start,  \
+                            seq_slots, out, ld_out, n_heads, qk_dim, v_dim, long_from)
+    if (dtype == SANDY_F32) { CASE(float, 1); CASE(float, 2); CASE(float, 3); CASE(float, 4); CASE(float, 6); CASE(float, 8); }
+    if (dtype == SANDY_BF16) { CASE(bf16, 1); CASE(bf16, 2); CASE(bf16, 3); CASE(bf16, 4); CASE(bf16, 6); CASE(bf16, 8); }
+#undef CASE
+    return SANDY_ERR_UNSUPPORTED;
+}
+
+// Floats of the chunked kernels' scratch for a step of n_tokens tokens of n_seqs requests: q, k, P, then the chunks' fading.
+SANDY_API long long sandy_gla_scratch_floats(int n_tokens, int n_seqs, int n_heads, int qk_dim) {
+    const long long dp = (qk_dim + 3) / 4 * 4;
+    return (long long)n_tokens * n_heads * (2 * dp + CC) + ((long long)n_tokens / CC + n_seqs + 1) * n_heads * dp;
+}
+
+// The chunked form, two launches, for requests that bring at least `long_from` tokens; max_q_len: the step's longest
+// portion.  scratch: float32, 16-byte aligned, as many floats as sandy_gla_scratch_floats says.
+SANDY_API int sandy_gla_chunk_scan(const void* proj, int ld, int dtype, int q_off, int k_off, int v_off, const float* low,
+                                   int ld_low, int rank, const float* w2t, const float* bias, float inv_tau, float q_scale,
+                                   float* state, long long state_stride, const int* q_start, const int* seq_slots, float* out,
+                                   int ld_out, float* scratch, int n_tokens, int n_seqs, int max_q_len, int n_heads, int qk_dim,
+                                   int v_dim, int long_from, cudaStream_t stream) {
+    if (n_seqs == 0 || n_tokens == 0) return SANDY_OK;
+    if (!proj || !low || !w2t || !bias || !state || !q_start || !seq_slots || !out || !scratch) return SANDY_ERR_ARGUMENT;
+    if (qk_dim <= 0 || qk_dim > MAX_DIM || v_dim <= 0 || n_heads <= 0 || n_heads > 65535 || n_seqs > 65535 || rank < 1 ||
+        rank > MAX_RANK || long_from < 1 || ((uintptr_t)scratch & 15))
+        return SANDY_ERR_UNSUPPORTED;
+    const long long dp = (qk_dim + 3) / 4 * 4;
+    float* qs = scratch;
+    float* ks = qs + (long long)n_tokens * n_heads * dp;
+    float* P = ks + (long long)n_tokens * n_heads * dp;
+    float* dec = P + (long long)n_tokens * n_heads * CC;
+    const dim3 grid_a((max_q_len + CC - 1) / CC, n_heads, n_seqs), grid_b(n_seqs, n_heads, (v_dim + COLS - 1) / COLS);
+    const size_t smem_a = prepare_smem(qk_dim, rank), smem_b = scan_smem(qk_dim);
+#define SCAN(TT, MAXR)                                                                                                    \
+    do {                                                                                                                  \
+        static size_t have_b = 0;                                                                                         \
+        if (int err = allow_smem(gla_chunk_scan_kernel<TT, MAXR>, smem_b, have_b)) return err;                            \
+        return sandy_launch(gla_chunk_scan_kernel<TT, MAXR>, grid_b, dim3(CT), smem_b, stream, (const TT*)proj, ld, v_off, \
+                            (const float*)qs, (const float*)ks, (const float*)P, (const float*)dec, state, state_stride,  \
+                            q_start, seq_slots, out, ld_out, n_heads, qk_dim, v_dim, long_from);                          \
+    } while (0)
+#define GO(TT)                                                                                                            \
+    do {                                                                                                                  \
+        static size_t have_a = 0;                                                                                         \
+        if (int err = allow_smem(gla_chunk_prepare_kernel<TT>, smem_a, have_a)) return err;                               \
+        if (int err = sandy_launch(gla_chunk_prepare_kernel<TT>, grid_a, dim3(CT), smem_a, stream, (const TT*)proj, ld,   \
+                                   q_off, k_off, low, ld_low, rank, w2t, bias, inv_tau, q_scale, q_start, qs, ks, P, dec, \
+                                   n_heads, qk_dim, long_from))                                                           \
+            return err;                                                                                                   \
+        if (qk_dim <= 32) SCAN(TT, 1);                                                                                    \
+        if (qk_dim <= 64) SCAN(TT, 2);                                                                                    \
+        if (qk_dim <= 128) SCAN(TT, 4);                                                                                   \
+        SCAN(TT, 8);                                                                                                      \
+    } while (0)
+    if (dtype == SANDY_F32) GO(float);
+    if (dtype == SANDY_BF16) GO(bf16);
+#undef GO
+#undef SCAN
+    return SANDY_ERR_UNSUPPORTED;
+}

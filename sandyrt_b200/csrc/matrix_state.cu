@@ -146,7 +146,10 @@ delta_scan_kernel(const float* __restrict__ qkv, int ld, const float* __restrict
     const int qh = h / (n_heads / n_qk_heads);
     const int per = per_token(d);
     const int t0 = q_start[s], t1 = q_start[s + 1];
-    if (long_from > 0 && t1 - t0 >= long_from) return;
+    if (long_from > 0 && t1 - t0 >= long_from) {
+        pdl_wait();                                   // a kernel ends only after the one before it has
+        return;
+    }
     float* S = state + (long long)seq_slots[s] * state_stride + (long long)h * e * d;    // [e][d]
     pdl_wait();
     float st[R][CPW];
@@ -258,7 +261,10 @@ mlstm_scan_kernel(const T* __restrict__ proj, int ld, int q_off, int k_off, int 
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const int per = per_token(d);
     const int t0 = q_start[s], t1 = q_start[s + 1];
-    if (long_from > 0 && t1 - t0 >= long_from) return;
+    if (long_from > 0 && t1 - t0 >= long_from) {
+        pdl_wait();                                   // a kernel ends only after the one before it has
+        return;
+    }
     float* base = state + (long long)seq_slots[s] * state_stride;
     float* S = base + (long long)h * e * d;
     float* n_st = base + (long long)n_heads * e * d + ((long long)h * Z + z) * d;
@@ -465,7 +471,10 @@ mlstm_chunk_kernel(const T* __restrict__ proj, int ld, int q_off, int k_off, int
     constexpr int MAXR = DPMAX / 32;
     const int s = blockIdx.x, h = blockIdx.y, z = blockIdx.z, col0 = z * COLS, Z = gridDim.z;
     const int t0 = q_start[s], t1 = q_start[s + 1];
-    if (t1 - t0 < long_from) return;
+    if (t1 - t0 < long_from) {
+        pdl_wait();
+        return;
+    }
     const int dp = (d + 3) / 4 * 4, ldq = dp + 4;
     const ChunkSmem m = carve(chunk_raw, dp, false);
     float* li = m.v1;     // a_j
@@ -649,7 +658,10 @@ delta_chunk_kernel(const float* __restrict__ qkv, int ld, const float* __restric
     constexpr int MAXR = DPMAX / 32;
     const int s = blockIdx.x, h = blockIdx.y, col0 = blockIdx.z * COLS;
     const int t0 = q_start[s], t1 = q_start[s + 1];
-    if (t1 - t0 < long_from) return;
+    if (t1 - t0 < long_from) {
+        pdl_wait();
+        return;
+    }
     const int qh = h / (n_heads / n_qk_heads);
     const int dp = (d + 3) / 4 * 4, ldq = dp + 4;
     const ChunkSmem m = carve(chunk_raw, dp, true);

@@ -9,6 +9,7 @@
 
 #include <cuda_runtime.h>
 
+#include "attention_rules.h"
 #include "matrix_state.h"
 
 #ifdef __cplusplus
@@ -182,6 +183,31 @@ int sandy_prefill_attention_tc_cap(const void* q, int ld_q, const void* k_cache,
                                    int head_dim, int page_size, float scale, int window, float softcap, int chunk,
                                    int num_pages, const float* sink, const float* out_gate, int* status, cudaStream_t stream);
 
+/* ... with everything of attention_rules.h that the kernel has a form for: also kept first keys behind a window and a gate
+   by element */
+int sandy_paged_attention_rules(const void* q, int ld_q, const void* k_cache, const void* v_cache, long long page_stride,
+                                const int* block_table, int max_blocks, const int* token_seq, const int* positions, void* out,
+                                int ld_out, int n_tokens, int n_heads, int n_kv_heads, int head_dim, int page_size, float scale,
+                                const SandyAttentionRules* rules, int num_pages, int dtype, int* status, cudaStream_t stream);
+int sandy_prefill_attention_rules(const void* q, int ld_q, const void* k_cache, const void* v_cache, long long page_stride,
+                                  const int* block_table, int max_blocks, const int* q_start, const int* kv_before, void* out,
+                                  int ld_out, int n_seqs, int max_q_len, int n_heads, int n_kv_heads, int head_dim, int page_size,
+                                  float scale, const SandyAttentionRules* rules, int num_pages, int* status, cudaStream_t stream);
+int sandy_prefill_attention_tc_rules(const void* q, int ld_q, const void* k_cache, const void* v_cache, long long page_stride,
+                                     const int* block_table, int max_blocks, const int* q_start, const int* kv_before, void* out,
+                                     int ld_out, int n_seqs, int max_q_len, int n_heads, int n_kv_heads, int head_dim, int page_size,
+                                     float scale, const SandyAttentionRules* rules, int num_pages, int* status, cudaStream_t stream);
+int sandy_decode_attention_shared_rules(const void* q, int ld_q, const void* k_cache, const void* v_cache, long long page_stride,
+                                        const int* block_table, int max_blocks, const int* token_seq, const int* positions, void* out,
+                                        int ld_out, int n_tokens, int n_heads, int n_kv_heads, int head_dim, int page_size, float scale,
+                                        const SandyAttentionRules* rules, int splits, int num_pages, float* scratch, int* status,
+                                        cudaStream_t stream);
+int sandy_decode_attention_mma_rules(const void* q, int ld_q, const void* k_cache, const void* v_cache, long long page_stride,
+                                     const int* block_table, int max_blocks, const int* token_seq, const int* positions, void* out,
+                                     int ld_out, int n_tokens, int n_heads, int n_kv_heads, int head_dim, int page_size, float scale,
+                                     const SandyAttentionRules* rules, int num_splits, int num_pages, int max_keys, int* status,
+                                     cudaStream_t stream);
+
 /* attention_decode_shared.cu */
 long long sandy_decode_attention_shared_scratch(int n_tokens, int n_heads, int n_kv_heads, int head_dim, int splits);
 int sandy_decode_attention_shared(const void* q, int ld_q, const void* k_cache, const void* v_cache, long long page_stride,
@@ -216,6 +242,27 @@ int sandy_attention_prepare_pos(const void* proj, int ld, int q_off, int k_off, 
                                 int ld_gate, float* gate_out, float gate_scale, const float* q_head_scale, float v_unit_eps,
                                 int per_head_norm, float q_pos_coef, int q_pos_every, int dtype, int* status,
                                 cudaStream_t stream);
+
+/* ... with the rotation's pairs chosen: interleaved != 0 pairs entries 2i and 2i + 1 */
+int sandy_attention_prepare_rot(const void* proj, int ld, int q_off, int k_off, int v_off, int n_tokens, int n_heads,
+                                int n_kv_heads, int qk_dim, int v_dim, int pad_dim, const float* q_gain, const float* k_gain,
+                                float eps, const float* freq, int rot_dims, const int* positions, const int* token_seq,
+                                const int* block_table, int max_blocks, void* k_cache, void* v_cache, long long page_stride,
+                                int page_size, int num_pages, int write_cache, void* q_out, int ld_q, const float* gate_in,
+                                int ld_gate, float* gate_out, float gate_scale, const float* q_head_scale, float v_unit_eps,
+                                int per_head_norm, float q_pos_coef, int q_pos_every, int interleaved, int dtype, int* status,
+                                cudaStream_t stream);
+
+/* gated_linear.cu */
+int sandy_gla_scan(const void* proj, int ld, int dtype, int q_off, int k_off, int v_off, const float* low, int ld_low, int rank,
+                   const float* w2t, const float* bias, float inv_tau, float q_scale, float* state, long long state_stride,
+                   const int* q_start, const int* seq_slots, float* out, int ld_out, int n_seqs, int n_heads, int qk_dim, int v_dim,
+                   int long_from, cudaStream_t stream);
+long long sandy_gla_scratch_floats(int n_tokens, int n_seqs, int n_heads, int qk_dim);
+int sandy_gla_chunk_scan(const void* proj, int ld, int dtype, int q_off, int k_off, int v_off, const float* low, int ld_low, int rank,
+                         const float* w2t, const float* bias, float inv_tau, float q_scale, float* state, long long state_stride,
+                         const int* q_start, const int* seq_slots, float* out, int ld_out, float* scratch, int n_tokens, int n_seqs,
+                         int max_q_len, int n_heads, int qk_dim, int v_dim, int long_from, cudaStream_t stream);
 
 /* rmsnorm.cu */
 int sandy_rmsnorm_shift(const float* x, int ldx, const float* gain, const float* mix, float* state, long long state_stride,
