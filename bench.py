@@ -8,6 +8,7 @@
     python bench.py --latent [--batch B]          Sovezen beside GPT-2 at equal layer sizes, likewise
     python bench.py --capped [--chunk N]          Bilurax beside Sovezen, likewise
     python bench.py --streams [--batch B]         Tifepel beside Panupel, likewise
+    python bench.py --linear [--window N]         Pugalix beside Panupel, likewise
     python bench.py --micro gemm|decode-attention|prefill-attention [...]   kernel micro-benchmarks
 
 Default workload: GPT-2 small (12 layers, width 768, 12 heads of 64, inner 3072, vocabulary 50257,
@@ -491,10 +492,27 @@ def streams_config(width, heads, kv_heads, ff, vocab=50257, layers=4):
             "layers": [{**(ssm if i % 2 == 0 else att), "mlp": moe} for i in range(layers)]}
 
 
-def hybrid(dtype_name: str, layers: int, batch: int, steps: int, warmup: int, design: str = "panupel", chunk: int = 1024) -> int:
-    """Prefill and decode throughput of a design (Panupel, Sovezen, Bilurax or Tifepel) at sizes that resemble real layers,
-    beside its closest relative with the same width, heads, layer count and vocabulary (GPT-2; for Bilurax, Sovezen; for
-    Tifepel, Panupel),
+# ---- windowed attention, gated linear attention and a matrix memory (Pugalix) beside Panupel at equal size ---------------
+# One of each in turn, the fourth layer attention on the first one's keys and values; heads of 64 on a third as many
+# key/value heads, a window of `window` positions behind 4 kept ones; gated linear attention with values twice as wide as
+# keys and a decay of rank 16; every layer with a feed-forward.
+def linear_config(width, heads, kv_heads, ff, vocab=50257, layers=4, window=512):
+    mask = {"size": window, "keep_first": 4}
+    att = {"type": "attention", "mixer": {"heads": heads, "kv_heads": kv_heads, "dim": 64, "vdim": 64, "scale": 0.125,
+                                          "rot": {"dims": 64, "base": 10000.0}, "mask": mask}}
+    gla = {"type": "gla", "mixer": {"heads": heads // 2, "dim": 64, "vdim": 128, "tau": 16.0, "rank": 16}}
+    mlstm = {"type": "mlstm", "mixer": {"heads": heads // 2, "dim": 64, "vdim": 128, "gate_cap": 12.0}}
+    reader = {"type": "attention", "mixer": {**att["mixer"], "kv_from": 0}}
+    kinds = [att, gla, mlstm, reader]
+    return {"architecture": "Pugalix", "vocab": vocab, "width": width, "embedding": {"scale": 1.0}, "norm": {"eps": 1e-6},
+            "layers": [{**kinds[i % 4], "mlp": {"kind": "dense", "ff": ff}} for i in range(layers)]}
+
+
+def hybrid(dtype_name: str, layers: int, batch: int, steps: int, warmup: int, design: str = "panupel", chunk: int = 1024,
+           window: int = 512) -> int:
+    """Prefill and decode throughput of a design (Panupel, Sovezen, Bilurax, Tifepel or Pugalix) at sizes that resemble real
+    layers, beside its closest relative with the same width, heads, layer count and vocabulary (GPT-2; for Bilurax, Sovezen;
+    for Tifepel and Pugalix, Panupel),
     both with random weights; then the device time per kernel class of both, so that like kernels can be held against
     each other.  One JSON line per size, then the tables."""
     import numpy as np
@@ -508,12 +526,13 @@ def hybrid(dtype_name: str, layers: int, batch: int, steps: int, warmup: int, de
     layers = layers or 4
     rng = np.random.default_rng(0)
     hybrid_config = {"panupel": globals()["hybrid_config"], "sovezen": latent_config,
-                     "bilurax": lambda **kw: capped_config(chunk=chunk, **kw), "tifepel": streams_config}[design]
+                     "bilurax": lambda **kw: capped_config(chunk=chunk, **kw), "tifepel": streams_config,
+                     "pugalix": lambda **kw: linear_config(window=window, **kw)}[design]
 
     def arms(sz):
         if design == "bilurax":
             return ((design, hybrid_config(layers=layers, **sz)), ("sovezen", latent_config(layers=layers, **sz)))
-        if design == "tifepel":
+        if design in ("tifepel", "pugalix"):
             return ((design, hybrid_config(layers=layers, **sz)), ("panupel", globals()["hybrid_config"](layers=layers, **sz)))
         gpt2_raw = {**load_model_config("small"), "n_embd": sz["width"], "n_head": sz["heads"], "n_inner": None, "n_layer": layers}
         return ((design, hybrid_config(layers=layers, **sz)), ("gpt2", gpt2_raw))
@@ -575,6 +594,10 @@ def main() -> int:
     ap.add_argument("--streams", action="store_true",
                     help="Tifepel (several copies of the stream around attention with a bias by distance and state-space layers, "
                          "routed experts) beside Panupel at equal sizes")
+    ap.add_argument("--linear", action="store_true",
+                    help="Pugalix (attention with a window that keeps the first tokens, gated linear attention, a matrix memory) "
+                         "beside Panupel at equal sizes")
+    ap.add_argument("--window", type=int, default=512, help="window of --linear")
     ap.add_argument("--micro", nargs=argparse.REMAINDER, help="run a kernel micro-benchmark (see sandyrt_b200/csrc/microbench.py)")
     args = ap.parse_args()
     if args.impl == "reference":
@@ -585,10 +608,10 @@ def main() -> int:
     if args.micro is not None:
         from sandyrt_b200.csrc import microbench
         return microbench.main(args.micro)
-    if args.hybrid or args.latent or args.capped or args.streams:
+    if args.hybrid or args.latent or args.capped or args.streams or args.linear:
         return hybrid(args.dtype, args.layers, args.batch, min(args.steps, 128), args.warmup,
-                      design="tifepel" if args.streams else "bilurax" if args.capped else "sovezen" if args.latent else "panupel",
-                      chunk=args.chunk)
+                      design="pugalix" if args.linear else "tifepel" if args.streams else "bilurax" if args.capped else
+                      "sovezen" if args.latent else "panupel", chunk=args.chunk, window=args.window)
     if args.workload:
         return workload(args.workload, args.dtype, args.layers)
     if args.profile_kernels:

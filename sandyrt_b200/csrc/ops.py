@@ -186,12 +186,37 @@ def kv_append(k_src, v_src, k_cache, v_cache, block_table, token_seq, positions)
     _check(code, "kv_append")
 
 
+class _AttentionRules(ctypes.Structure):
+    """SandyAttentionRules of attention_rules.h."""
+    _fields_ = [("window", ctypes.c_int), ("keep_first", ctypes.c_int), ("softcap", ctypes.c_float), ("chunk", ctypes.c_int),
+                ("sink", ctypes.c_void_p), ("out_gate", ctypes.c_void_p), ("dist_bias", ctypes.c_void_p), ("n_dist", ctypes.c_int),
+                ("elem_gate", ctypes.c_void_p), ("ld_elem_gate", ctypes.c_int), ("gate_dim", ctypes.c_int)]
+
+
+def _rules(q, n_heads: int, window=0, keep_first=0, softcap=0.0, chunk=0, sink=None, out_gate=None, dist_bias=None, elem_gate=None):
+    """The rules as the kernels take them.  elem_gate: [T, H * dim] of q's type, any row pitch."""
+    _cuda(sink, out_gate, dist_bias, elem_gate)
+    if dist_bias is not None and (dist_bias.dtype != torch.float32 or dist_bias.dim() != 2 or dist_bias.shape[0] != n_heads
+                                  or not dist_bias.is_contiguous()):
+        raise KernelError("attention: a bias by distance is a dense float32 [H, n_dist]")
+    if elem_gate is not None and (elem_gate.dtype != q.dtype or elem_gate.shape[0] != q.shape[0] or elem_gate.shape[1] % n_heads
+                                  or elem_gate.shape[1] > q.shape[1] or elem_gate.stride(1) != 1):
+        raise KernelError("attention: a gate by element is [T, H * dim] of the queries' type")
+    ptr = lambda t: None if t is None else t.data_ptr()
+    return ctypes.byref(_AttentionRules(window, keep_first, softcap, chunk, ptr(sink), ptr(out_gate), ptr(dist_bias),
+                                        0 if dist_bias is None else dist_bias.shape[1], ptr(elem_gate),
+                                        0 if elem_gate is None else elem_gate.stride(0),
+                                        0 if elem_gate is None else elem_gate.shape[1] // n_heads))
+
+
 def paged_attention(q, k_cache, v_cache, block_table, token_seq, positions, out, *, sink=None, out_gate=None,
-                    n_heads: int, scale: float, window: int = 0, softcap: float = 0.0, chunk: int = 0, dist_bias=None) -> None:
+                    n_heads: int, scale: float, window: int = 0, softcap: float = 0.0, chunk: int = 0, dist_bias=None,
+                    keep_first: int = 0, elem_gate=None) -> None:
     """Causal attention of every token of the step over its request's pages (general kernel).  softcap > 0 presses
     every score into softcap * tanh(score / softcap); chunk > 0 lets a query see the keys of its own chunk of
     positions only; dist_bias (float32 [H, n_dist]) adds entry min(i - j, n_dist - 1) of the head's row to the score of
-    query i and key j."""
+    query i and key j; keep_first leaves keys 0 .. keep_first - 1 visible behind a window; elem_gate ([T, H * dim] of q's
+    type) multiplies entry i < dim of a head's output by sigmoid of its own."""
     _cuda(q, k_cache, v_cache, block_table, token_seq, positions, out)
     hkv, ps, d, page_stride, num_pages = _cache_args(k_cache, v_cache)
     T = q.shape[0]
@@ -204,23 +229,14 @@ def paged_attention(q, k_cache, v_cache, block_table, token_seq, positions, out,
         raise KernelError("attention: q and out must be [T, H*D] of the cache's dtype")
     _i32(block_table, "block_table"); _i32(token_seq, "token_seq"); _i32(positions, "positions")
     lib = load_library("attention")
-    code = lib.sandy_paged_attention_bias(_p(q), ctypes.c_int(q.stride(0)), _p(k_cache), _p(v_cache),
+    rules = _rules(q, n_heads, window, keep_first, softcap, chunk, sink, out_gate, dist_bias, elem_gate)
+    code = lib.sandy_paged_attention_rules(_p(q), ctypes.c_int(q.stride(0)), _p(k_cache), _p(v_cache),
                                      ctypes.c_longlong(page_stride), _p(block_table),
                                      ctypes.c_int(block_table.shape[1]), _p(token_seq), _p(positions), _p(out),
                                      ctypes.c_int(out.stride(0)), ctypes.c_int(T), ctypes.c_int(n_heads),
-                                     ctypes.c_int(hkv), ctypes.c_int(d), ctypes.c_int(ps), ctypes.c_float(scale),
-                                     ctypes.c_int(window), ctypes.c_float(softcap), ctypes.c_int(chunk),
-                                     ctypes.c_int(num_pages), ctypes.c_int(_dt(q)),
-                                     _p(sink), _p(out_gate), *_bias_args(dist_bias, n_heads), _p(kernel_status(q.device)), _stream())
+                                     ctypes.c_int(hkv), ctypes.c_int(d), ctypes.c_int(ps), ctypes.c_float(scale), rules,
+                                     ctypes.c_int(num_pages), ctypes.c_int(_dt(q)), _p(kernel_status(q.device)), _stream())
     _check(code, f"paged_attention(H={n_heads},Hkv={hkv},D={d})")
-
-
-def _bias_args(dist_bias, n_heads: int):
-    if dist_bias is None:
-        return None, ctypes.c_int(0)
-    if dist_bias.dtype != torch.float32 or dist_bias.dim() != 2 or dist_bias.shape[0] != n_heads or not dist_bias.is_contiguous():
-        raise KernelError("attention: a bias by distance is a dense float32 [H, n_dist]")
-    return _p(dist_bias), ctypes.c_int(dist_bias.shape[1])
 
 
 _DECODE_HEAD_DIMS = {torch.bfloat16: (16, 32, 64, 128, 256), torch.float32: (16, 32, 64, 128)}
@@ -240,13 +256,16 @@ CLUSTER_MAX_SPLITS = 8
 
 def decode_attention(q, k_cache, v_cache, block_table, token_seq, positions, out, *, n_heads: int,
                      scale: float, window: int = 0, num_splits: int = 1, scratch=None, cluster: bool = False,
-                     bulk: bool = False, mma: bool = False, sink=None, out_gate=None) -> None:
+                     bulk: bool = False, mma: bool = False, sink=None, out_gate=None, keep_first: int = 0, elem_gate=None) -> None:
     """Split-KV attention of single tokens (head sizes 16/32/64/128, 256 in bfloat16).  With
     `cluster` (2..8 splits) the splits merge through distributed shared memory inside one
     kernel; otherwise they go through `scratch` and a merge kernel.  `bulk` (at most 8 splits)
     runs the variant that streams whole pages into shared memory with bulk copies, which is
     the faster one when there are hundreds of (token, head) pairs.  `mma` (bfloat16, heads of 64, at
-    most 8 splits) runs the variant whose products are mma.sync instructions."""
+    most 8 splits) runs the variant whose products are mma.sync instructions, the only one here with a form for
+    keep_first and elem_gate (as in paged_attention)."""
+    if (keep_first or elem_gate is not None) and not mma:
+        raise UnsupportedShape("decode_attention: kept first keys and a gate by element need the mma.sync kernel")
     _cuda(q, k_cache, v_cache, block_table, token_seq, positions, out, scratch)
     hkv, ps, d, page_stride, num_pages = _cache_args(k_cache, v_cache)
     T = q.shape[0]
@@ -264,12 +283,13 @@ def decode_attention(q, k_cache, v_cache, block_table, token_seq, positions, out
         if num_splits > CLUSTER_MAX_SPLITS:
             raise UnsupportedShape(f"decode_attention: a cluster holds at most {CLUSTER_MAX_SPLITS} splits")
         lib = load_library("attention_decode_mma")
-        code = lib.sandy_decode_attention_mma_ext(
+        code = lib.sandy_decode_attention_mma_rules(
             _p(q), ctypes.c_int(q.stride(0)), _p(k_cache), _p(v_cache), ctypes.c_longlong(page_stride),
             _p(block_table), ctypes.c_int(block_table.shape[1]), _p(token_seq), _p(positions), _p(out),
             ctypes.c_int(out.stride(0)), ctypes.c_int(T), ctypes.c_int(n_heads), ctypes.c_int(hkv), ctypes.c_int(d),
-            ctypes.c_int(ps), ctypes.c_float(scale), ctypes.c_int(window), ctypes.c_int(num_splits),
-            ctypes.c_int(num_pages), ctypes.c_int(block_table.shape[1] * ps), _p(sink), _p(out_gate), _p(kernel_status(q.device)), _stream())
+            ctypes.c_int(ps), ctypes.c_float(scale),
+            _rules(q, n_heads, window, keep_first, sink=sink, out_gate=out_gate, elem_gate=elem_gate), ctypes.c_int(num_splits),
+            ctypes.c_int(num_pages), ctypes.c_int(block_table.shape[1] * ps), _p(kernel_status(q.device)), _stream())
         _check(code, f"decode_attention_mma(H={n_heads},Hkv={hkv},page={ps},splits={num_splits})")
         return
     if bulk:
@@ -315,9 +335,11 @@ def decode_attention(q, k_cache, v_cache, block_table, token_seq, positions, out
 
 
 def decode_attention_shared(q, k_cache, v_cache, block_table, token_seq, positions, out, *, n_heads: int, scale: float, splits: int = 1,
-                            window: int = 0, sink=None, out_gate=None, softcap: float = 0.0, chunk: int = 0, dist_bias=None) -> None:
+                            window: int = 0, sink=None, out_gate=None, softcap: float = 0.0, chunk: int = 0, dist_bias=None,
+                            keep_first: int = 0, elem_gate=None) -> None:
     """Single-token attention with the query heads of a group as the rows of one tensor-core product (bfloat16, head sizes
-    up to 128); v_cache may be k_cache itself (one plane).  softcap, chunk and dist_bias as in paged_attention."""
+    up to 128); v_cache may be k_cache itself (one plane).  softcap, chunk, dist_bias, keep_first and elem_gate as in
+    paged_attention."""
     _cuda(q, k_cache, v_cache, block_table, token_seq, positions, out)
     hkv, ps, d, page_stride, num_pages = _cache_args(k_cache, v_cache)
     T = q.shape[0]
@@ -325,23 +347,24 @@ def decode_attention_shared(q, k_cache, v_cache, block_table, token_seq, positio
     lib.sandy_decode_attention_shared_scratch.restype = ctypes.c_longlong
     floats = lib.sandy_decode_attention_shared_scratch(ctypes.c_int(T), ctypes.c_int(n_heads), ctypes.c_int(hkv), ctypes.c_int(d), ctypes.c_int(splits))
     scratch = torch.empty(max(int(floats), 1), dtype=torch.float32, device=q.device)
-    code = lib.sandy_decode_attention_shared_bias(
+    code = lib.sandy_decode_attention_shared_rules(
         _p(q), ctypes.c_int(q.stride(0)), _p(k_cache), _p(v_cache), ctypes.c_longlong(page_stride), _p(block_table),
         ctypes.c_int(block_table.shape[1]), _p(token_seq), _p(positions), _p(out), ctypes.c_int(out.stride(0)), ctypes.c_int(T),
-        ctypes.c_int(n_heads), ctypes.c_int(hkv), ctypes.c_int(d), ctypes.c_int(ps), ctypes.c_float(scale), ctypes.c_int(window),
-        ctypes.c_float(softcap), ctypes.c_int(chunk), ctypes.c_int(splits), ctypes.c_int(num_pages), _p(sink), _p(out_gate),
-        *_bias_args(dist_bias, n_heads), _p(scratch), _p(kernel_status(q.device)), _stream())
+        ctypes.c_int(n_heads), ctypes.c_int(hkv), ctypes.c_int(d), ctypes.c_int(ps), ctypes.c_float(scale),
+        _rules(q, n_heads, window, keep_first, softcap, chunk, sink, out_gate, dist_bias, elem_gate), ctypes.c_int(splits),
+        ctypes.c_int(num_pages), _p(scratch), _p(kernel_status(q.device)), _stream())
     _check(code, f"decode_attention_shared(H={n_heads},Hkv={hkv},D={d})")
 
 
 def prefill_attention(q, k_cache, v_cache, block_table, q_start, kv_before, out, *, sink=None, out_gate=None, n_heads: int,
                       max_q_len: int, scale: float, window: int = 0, tc=None, softcap: float = 0.0, chunk: int = 0,
-                      dist_bias=None) -> None:
+                      dist_bias=None, keep_first: int = 0, elem_gate=None) -> None:
     """Tensor-core attention of prompt portions (bfloat16, head sizes 16..128 in steps of 16).
     q_start: int32 [S+1] first new token of each request; kv_before: int32 [S].
     tc: True asks for the tcgen05 kernel (heads of 64), False for the mma.sync kernel, None
     picks the tcgen05 kernel where it takes the shape.  softcap and chunk as in paged_attention; both kernels
-    have the form for them.  dist_bias as in paged_attention: the mma.sync kernel alone has the form for it."""
+    have the form for them.  dist_bias as in paged_attention: the mma.sync kernel alone has the form for it.  keep_first and
+    elem_gate as in paged_attention, in both kernels."""
     _cuda(q, k_cache, v_cache, block_table, q_start, kv_before, out, sink, out_gate)
     hkv, ps, d, page_stride, num_pages = _cache_args(k_cache, v_cache)
     if q.dtype != torch.bfloat16 or d % 16 != 0 or d > 128:
@@ -358,25 +381,18 @@ def prefill_attention(q, k_cache, v_cache, block_table, q_start, kv_before, out,
     args = (_p(q), ctypes.c_int(q.stride(0)), _p(k_cache), _p(v_cache), ctypes.c_longlong(page_stride),
             _p(block_table), ctypes.c_int(block_table.shape[1]), _p(q_start), _p(kv_before), _p(out),
             ctypes.c_int(out.stride(0)), ctypes.c_int(S), ctypes.c_int(max_q_len), ctypes.c_int(n_heads),
-            ctypes.c_int(hkv), ctypes.c_int(d), ctypes.c_int(ps), ctypes.c_float(scale), ctypes.c_int(window),
-            ctypes.c_float(softcap), ctypes.c_int(chunk),
-            ctypes.c_int(num_pages), _p(sink), _p(out_gate), _p(kernel_status(q.device)), _stream())
+            ctypes.c_int(hkv), ctypes.c_int(d), ctypes.c_int(ps), ctypes.c_float(scale),
+            _rules(q, n_heads, window, keep_first, softcap, chunk, sink, out_gate, dist_bias, elem_gate),
+            ctypes.c_int(num_pages), _p(kernel_status(q.device)), _stream())
     if dist_bias is not None and tc:
         raise UnsupportedShape("prefill_attention: the tcgen05 kernel takes no bias by distance")
     if tc or (tc is None and d == 64 and dist_bias is None):
-        code = load_library("attention_prefill_tc").sandy_prefill_attention_tc_cap(*args)
+        code = load_library("attention_prefill_tc").sandy_prefill_attention_tc_rules(*args)
         if code != -1 or tc:
             _check(code, f"prefill_attention_tc(H={n_heads},Hkv={hkv},D={d})")
             return
     lib = load_library("attention_prefill")
-    code = lib.sandy_prefill_attention_bias(_p(q), ctypes.c_int(q.stride(0)), _p(k_cache), _p(v_cache),
-                                       ctypes.c_longlong(page_stride), _p(block_table),
-                                       ctypes.c_int(block_table.shape[1]), _p(q_start), _p(kv_before), _p(out),
-                                       ctypes.c_int(out.stride(0)), ctypes.c_int(S), ctypes.c_int(max_q_len),
-                                       ctypes.c_int(n_heads), ctypes.c_int(hkv), ctypes.c_int(d), ctypes.c_int(ps),
-                                       ctypes.c_float(scale), ctypes.c_int(window), ctypes.c_float(softcap),
-                                       ctypes.c_int(chunk), ctypes.c_int(num_pages),
-                                       _p(sink), _p(out_gate), *_bias_args(dist_bias, n_heads), _p(kernel_status(q.device)), _stream())
+    code = lib.sandy_prefill_attention_rules(*args)
     _check(code, f"prefill_attention(H={n_heads},Hkv={hkv},D={d})")
 
 
@@ -725,6 +741,43 @@ def gated_group_norm(y, z, gain, out, *, groups: int, eps: float) -> None:
         _p(y), ctypes.c_int(y.stride(0)), _p(z), ctypes.c_int(z.stride(0)), _p(gain), ctypes.c_float(eps), ctypes.c_int(groups), _p(out),
         ctypes.c_int(out.stride(0)), ctypes.c_int(y.shape[0]), ctypes.c_int(y.shape[1]), ctypes.c_int(_dt(out)), _stream())
     _check(code, "gated_group_norm")
+
+
+def attention_prepare(proj, k_cache, v_cache, block_table, token_seq, positions, q_out, *, n_heads: int, qk_dim: int, v_dim: int,
+                      freq=None, interleaved: bool = False, write_cache: bool = True) -> None:
+    """Queries, keys and values out of a projection [T, H * qk_dim | Hkv * qk_dim | Hkv * v_dim | ...]: the first
+    2 * len(freq) entries of every query and key head turn (halves, or neighbours with `interleaved`), keys and values go
+    into their pages, queries into q_out [T, H * D], heads padded with zeros to the cache's head size D."""
+    _cuda(proj, k_cache, v_cache, block_table, token_seq, positions, q_out, freq)
+    hkv, ps, d, page_stride, num_pages = _cache_args(k_cache, v_cache)
+    null, i = ctypes.c_void_p(0), ctypes.c_int
+    code = load_library("attention_prepare").sandy_attention_prepare_rot(
+        _p(proj), i(proj.stride(0)), i(0), i(n_heads * qk_dim), i((n_heads + hkv) * qk_dim), i(proj.shape[0]), i(n_heads), i(hkv), i(qk_dim),
+        i(v_dim), i(d), null, null, ctypes.c_float(0.0), _p(freq), i(0 if freq is None else 2 * freq.numel()), _p(positions), _p(token_seq),
+        _p(block_table), i(block_table.shape[1]), _p(k_cache), _p(v_cache), ctypes.c_longlong(page_stride), i(ps), i(num_pages),
+        i(1 if write_cache else 0), _p(q_out), i(q_out.stride(0)), null, i(0), null, ctypes.c_float(1.0), null, ctypes.c_float(0.0), i(0),
+        ctypes.c_float(0.0), i(0), i(1 if interleaved else 0), i(_dt(proj)), _p(kernel_status(proj.device)), _stream())
+    _check(code, "attention_prepare")
+
+
+def gla_scan(proj, low, w2t, bias, state, q_start, seq_slots, out, *, n_heads: int, qk_dim: int, v_dim: int, tau: float,
+             q_scale: float, chunked_from: int = 0, max_q_len: int = 0) -> None:
+    """Gated linear attention: S <- diag(alpha) S + k v^T per head, out = S^T (q q_scale), alpha = sigmoid(low w2t + bias)^(1 / tau).
+    proj [T, H * qk_dim | H * qk_dim | H * v_dim | ...] (q, k, v); low float32 [T, rank]; w2t float32 [rank, H * qk_dim]; `state`
+    float32 [slots, >= H * v_dim * qk_dim].  Requests with chunked_from tokens or more take the chunked kernels (0: none)."""
+    _cuda(proj, low, w2t, bias, state, q_start, seq_slots, out)
+    lib, i, f = load_library("gated_linear"), ctypes.c_int, ctypes.c_float
+    S, T = seq_slots.numel(), proj.shape[0]
+    head = (_p(proj), i(proj.stride(0)), i(_dt(proj)), i(0), i(n_heads * qk_dim), i(2 * n_heads * qk_dim), _p(low), i(low.stride(0)),
+            i(low.shape[1]), _p(w2t), _p(bias), f(1.0 / tau), f(q_scale), _p(state), ctypes.c_longlong(state.stride(0)), _p(q_start),
+            _p(seq_slots), _p(out), i(out.stride(0)))
+    _check(lib.sandy_gla_scan(*head, i(S), i(n_heads), i(qk_dim), i(v_dim), i(chunked_from), _stream()), "gla_scan")
+    if chunked_from:
+        lib.sandy_gla_scratch_floats.restype = ctypes.c_longlong
+        floats = lib.sandy_gla_scratch_floats(i(T), i(S), i(n_heads), i(qk_dim))
+        scratch = torch.full((int(floats),), float("nan"), dtype=torch.float32, device=proj.device)
+        _check(lib.sandy_gla_chunk_scan(*head, _p(scratch), i(T), i(S), i(max_q_len), i(n_heads), i(qk_dim), i(v_dim), i(chunked_from),
+                                        _stream()), "gla_chunk_scan")
 
 
 def sample(logits, out_tokens, *, temperature=None, top_k=None, top_p=None, uniform=None, status=None,
