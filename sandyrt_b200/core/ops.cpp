@@ -142,15 +142,15 @@ void spin(cudaStream_t stream, long long nanoseconds) {
 }
 
 void embed_positions(const Launch& l, const int* ids, const int* positions, const Tensor& wte, const Tensor* wpe, Tensor& out,
-                     int n_tokens) {
+                     int n_tokens, float scale) {
     if (wpe && (wpe->dtype != wte.dtype || wpe->cols != out.cols))
         throw KernelError("position table must match the token table in dtype and width");
     if (wte.cols != out.cols || !wte.contiguous() || !out.contiguous() || out.rows < n_tokens)
         throw KernelError("embed_positions: tables and output must be contiguous and of one width");
-    static auto fn = SANDY_KERNEL(embed, sandy_embed_pos);
+    static auto fn = SANDY_KERNEL(embed, sandy_embed_pos_scaled);
     OpTimer timer(l, "embedding", (double)n_tokens * out.cols * ((wpe ? 2.0 : 1.0) * wte.elem_size() + out.elem_size()), 0);
     check(fn(ids, positions, wte.data, wpe ? wpe->data : nullptr, out.data, n_tokens, (int)out.cols, (int)wte.rows,
-             wpe ? (int)wpe->rows : 0, code_of(wte.dtype), code_of(out.dtype), l.status, l.stream),
+             wpe ? (int)wpe->rows : 0, scale, code_of(wte.dtype), code_of(out.dtype), l.status, l.stream),
           "embed_positions");
 }
 

@@ -49,8 +49,9 @@ std::vector<ProfileRow> profile_report();              // also clears what was g
 int sm_count();                                        // streaming multiprocessors of the current device
 void spin(cudaStream_t stream, long long nanoseconds); // keeps the stream busy (timing loops queue launches behind it)
 
+// out[t] = (wte[ids[t]] + wpe[positions[t]]) * scale; wpe may be null.
 void embed_positions(const Launch& l, const int* ids, const int* positions, const Tensor& wte, const Tensor* wpe,
-                     Tensor& out, int n_tokens);
+                     Tensor& out, int n_tokens, float scale = 1.0f);
 void layernorm(const Launch& l, const Tensor& x, const Tensor& gamma, const Tensor* beta, float eps, Tensor& out,
                const int* rows, int n_rows);
 
@@ -124,8 +125,8 @@ struct AttentionStep {
     const int* kv_before = nullptr;
     const int* block_table = nullptr;
     int max_blocks = 0;
-    // from the step's host-side lists, for the profile's figures only: keys the step's requests hold
-    // after it, and (query, key) pairs the causal attention looks at
+    // from the step's host-side lists, for the profile's figures only: keys of the step's requests that are
+    // read, and (query, key) pairs the causal attention looks at
     double kv_tokens = 0, pairs = 0;
 };
 // What some attention layers add to the softmax: a sink per head (float32 [H]: exp(sink) joins the denominator and

@@ -1,10 +1,11 @@
 #include "parts.h"
 
+#include <algorithm>
 #include <mutex>
 
 namespace sandy {
 
-ops::AttentionStep StepContext::attention_step(int group) const {
+ops::AttentionStep StepContext::attention_step(int group, int window, int keep_first) const {
     ops::AttentionStep s;
     s.n_tokens = n_tokens;
     s.n_seqs = n_seqs;
@@ -17,6 +18,12 @@ ops::AttentionStep StepContext::attention_step(int group) const {
     s.max_blocks = max_blocks;
     for (size_t i = 0; i < host_q_lens.size() && i < host_kv_before.size(); i++) {
         const double n = host_q_lens[i], before = host_kv_before[i];
+        if (window > 0) {
+            const int most = window + keep_first;
+            s.kv_tokens += std::min(before + n, most + n - 1);
+            for (int k = host_kv_before[i] + 1; k <= host_kv_before[i] + host_q_lens[i]; k++) s.pairs += std::min(k, most);
+            continue;
+        }
         s.kv_tokens += before + n;
         s.pairs += n * before + n * (n + 1) / 2;
     }
@@ -206,8 +213,7 @@ public:
     const Tensor* table() const override { return &weight_.view; }
     void forward(StepContext& ctx, Tensor& x) override {
         const Tensor* pos = ctx.position ? ctx.position->table() : nullptr;
-        ops::embed_positions(ctx.launch, ctx.token_ids, ctx.positions, weight_.view, pos, x, ctx.n_tokens);
-        if (scale_ != 1.0f) ops::scale(ctx.launch, x, scale_);
+        ops::embed_positions(ctx.launch, ctx.token_ids, ctx.positions, weight_.view, pos, x, ctx.n_tokens, scale_);
     }
 private:
     int64_t vocab_, width_;

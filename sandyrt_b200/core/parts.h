@@ -78,7 +78,8 @@ struct StepContext {
     int max_q_len = 0, max_kv_len = 0;
     ops::Launch launch;                  // stream and status words
 
-    ops::AttentionStep attention_step(int group) const;
+    // `window` and `keep_first` of the layer that asks: the profile's figures count the keys it looks at
+    ops::AttentionStep attention_step(int group, int window = 0, int keep_first = 0) const;
 };
 
 class Part {

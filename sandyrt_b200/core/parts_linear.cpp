@@ -130,7 +130,7 @@ public:
             gate = wide.col_range(n_wide_ - (int64_t)H_ * e_, n_wide_);
             extras.elem_gate = &gate;
         }
-        ops::attention(l, ctx.attention_step(cache.group), q, cache, heads, H_, scale_, window_, ws, &extras);
+        ops::attention(l, ctx.attention_step(cache.group, window_, keep_), q, cache, heads, H_, scale_, window_, ws, &extras);
         out_.run(ctx, nullptr, &heads, x, ops::Act::None, ctx.overwrite ? nullptr : &x);
     }
 private:

@@ -1,6 +1,6 @@
 // Token embedding with the learned position table added in the same pass.
 //
-//   x[t, :] = wte[id[t], :] + wpe[pos[t], :]
+//   x[t, :] = (wte[id[t], :] + wpe[pos[t], :]) * scale
 //
 // The reference runs two gathers and an add (src/models/gpt2_small.sandy.go:48-50;
 // gather kernel src/device/cuda/CudaGatherKernels.cu:97-117, one thread per element).
@@ -14,7 +14,7 @@ template <typename TT, typename TO>
 __global__ void embed_pos_kernel(const int* __restrict__ ids, const int* __restrict__ pos,
                                  const TT* __restrict__ wte, const TT* __restrict__ wpe,
                                  TO* __restrict__ out, int width, int vocab, int n_pos,
-                                 int* __restrict__ status) {
+                                 float scale, int* __restrict__ status) {
     // The first kernel of a step lets its successors start only after its own wait has returned: by then
     // every kernel of the steps before has completed, so the step's later kernels may read what those steps
     // wrote (cache pages of older positions, the index arrays) before their own waits.
@@ -34,26 +34,33 @@ __global__ void embed_pos_kernel(const int* __restrict__ ids, const int* __restr
             v = to_f32(trow[e]);
             if (prow) v += to_f32(prow[e]);
         }
-        orow[e] = from_f32<TO>(v);
+        orow[e] = from_f32<TO>(v * scale);
     }
 }
 
 // ids, pos: int32[n_tokens]; wte: [vocab, width]; wpe: [n_pos, width] or null (no table);
 // out: [n_tokens, width].  status: device int, bit 0 = bad token id, bit 1 = bad position.
-SANDY_API int sandy_embed_pos(const int* ids, const int* pos, const void* wte, const void* wpe,
-                              void* out, int n_tokens, int width, int vocab, int n_pos,
-                              int table_dtype, int out_dtype, int* status, cudaStream_t stream) {
+SANDY_API int sandy_embed_pos_scaled(const int* ids, const int* pos, const void* wte, const void* wpe,
+                                     void* out, int n_tokens, int width, int vocab, int n_pos, float scale,
+                                     int table_dtype, int out_dtype, int* status, cudaStream_t stream) {
     if (n_tokens == 0) return SANDY_OK;
     if (!ids || !wte || !out || width <= 0) return SANDY_ERR_ARGUMENT;
     const int threads = width >= 1024 ? 256 : (width >= 256 ? 128 : 64);
 #define LAUNCH(TT, TO)                                                                          \
     return sandy_launch(embed_pos_kernel<TT, TO>, dim3(n_tokens), dim3(threads), 0, stream, ids, pos,  \
-                        (const TT*)wte, (const TT*)wpe, (TO*)out, width, vocab, n_pos, status)
+                        (const TT*)wte, (const TT*)wpe, (TO*)out, width, vocab, n_pos, scale, status)
     if (table_dtype == SANDY_F32 && out_dtype == SANDY_F32) LAUNCH(float, float);
     if (table_dtype == SANDY_BF16 && out_dtype == SANDY_F32) LAUNCH(bf16, float);
     if (table_dtype == SANDY_BF16 && out_dtype == SANDY_BF16) LAUNCH(bf16, bf16);
 #undef LAUNCH
     return SANDY_ERR_UNSUPPORTED;
+}
+
+// The same with a scale of one.
+SANDY_API int sandy_embed_pos(const int* ids, const int* pos, const void* wte, const void* wpe,
+                              void* out, int n_tokens, int width, int vocab, int n_pos,
+                              int table_dtype, int out_dtype, int* status, cudaStream_t stream) {
+    return sandy_embed_pos_scaled(ids, pos, wte, wpe, out, n_tokens, width, vocab, n_pos, 1.0f, table_dtype, out_dtype, status, stream);
 }
 
 // ---- small device utilities the host side uses -------------------------------------------------

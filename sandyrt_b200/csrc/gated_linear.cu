@@ -303,7 +303,7 @@ gla_chunk_scan_kernel(const T* __restrict__ proj, int ld, int v_off, const float
         const int c = x / dp, i = x % dp;            // consecutive threads read consecutive rows of a column
         S0[i * COLS + c] = (i < d && col0 + c < e) ? S[(size_t)(col0 + c) * d + i] : 0.0f;
     }
-    float pre_v[CC * COLS / CT];
+    T pre_v[CC * COLS / CT];                         // as loaded: a conversion here would make the warp wait for it
     auto fetch = [&](int tc, int b) {                // chunk at token tc into buffer b; nothing behind the last token
         float* dst = buf + b * buf_floats;
         const int n_tok = t1 - tc, pieces = dp / 4;
@@ -325,7 +325,9 @@ gla_chunk_scan_kernel(const T* __restrict__ proj, int ld, int v_off, const float
 #pragma unroll
         for (int u = 0; u < CC * COLS / CT; u++) {
             const int x = tid + u * CT, t = x / COLS, c = x % COLS;
-            pre_v[u] = (t < n_tok && col0 + c < e) ? to_f32(proj[(size_t)(tc + t) * ld + v_off + h * e + col0 + c]) : 0.0f;
+            T v = from_f32<T>(0.0f);
+            if (t < n_tok && col0 + c < e) v = proj[(size_t)(tc + t) * ld + v_off + h * e + col0 + c];
+            pre_v[u] = v;
         }
     };
     const int ot = tid / 8, oc = (tid % 8) * 2;      // this thread's token (and first state row) and two columns
@@ -334,7 +336,7 @@ gla_chunk_scan_kernel(const T* __restrict__ proj, int ld, int v_off, const float
         const int n_tok = min(CC, t1 - tc);
         __syncthreads();                             // everyone is done with sv and the other buffer
 #pragma unroll
-        for (int u = 0; u < CC * COLS / CT; u++) sv[tid + u * CT] = pre_v[u];
+        for (int u = 0; u < CC * COLS / CT; u++) sv[tid + u * CT] = to_f32(pre_v[u]);
         const bool more = tc + CC < t1;
         if (more) fetch(tc + CC, b ^ 1);
         if (more) asm volatile("cp.async.wait_group 1;" ::: "memory");
@@ -347,6 +349,7 @@ gla_chunk_scan_kernel(const T* __restrict__ proj, int ld, int v_off, const float
         float o[2] = {0.0f, 0.0f};
         {
             const float* qrow = q + ot * dp;
+#pragma unroll 4
             for (int i = 0; i < dp; i += 4) {
                 const float4 x = *reinterpret_cast<const float4*>(qrow + i);
                 const float2 a0 = *reinterpret_cast<const float2*>(S0 + (i + 0) * COLS + oc), a1 = *reinterpret_cast<const float2*>(S0 + (i + 1) * COLS + oc);
@@ -357,6 +360,7 @@ gla_chunk_scan_kernel(const T* __restrict__ proj, int ld, int v_off, const float
                 o[0] = fmaf(x.w, a3.x, o[0]); o[1] = fmaf(x.w, a3.y, o[1]);
             }
             const float* prow = p + ot * CC;
+#pragma unroll 2
             for (int j = 0; j <= ot; j += 4) {       // P is zero behind the diagonal, v behind the last token
                 const float4 x = *reinterpret_cast<const float4*>(prow + j);
                 const float2 a0 = *reinterpret_cast<const float2*>(sv + (j + 0) * COLS + oc), a1 = *reinterpret_cast<const float2*>(sv + (j + 1) * COLS + oc);
@@ -382,7 +386,8 @@ gla_chunk_scan_kernel(const T* __restrict__ proj, int ld, int v_off, const float
                 sn[r][0] = f * x.x; sn[r][1] = f * x.y;
             }
         }
-        for (int j = 0; j < n_tok; j++) {
+#pragma unroll 8
+        for (int j = 0; j < CC; j++) {               // k and v are zero behind the last token
             const float2 v = *reinterpret_cast<const float2*>(sv + j * COLS + oc);
 #pragma unroll
             for (int r = 0; r < MAXR; r++) {

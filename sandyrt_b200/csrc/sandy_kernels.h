@@ -19,6 +19,8 @@ extern "C" {
 /* embed.cu */
 int sandy_embed_pos(const int* ids, const int* pos, const void* wte, const void* wpe, void* out, int n_tokens, int width,
                     int vocab, int n_pos, int table_dtype, int out_dtype, int* status, cudaStream_t stream);
+int sandy_embed_pos_scaled(const int* ids, const int* pos, const void* wte, const void* wpe, void* out, int n_tokens, int width,
+                           int vocab, int n_pos, float scale, int table_dtype, int out_dtype, int* status, cudaStream_t stream);
 int sandy_device_sm_count(void);
 int sandy_spin(long long nanoseconds, cudaStream_t stream);
 
