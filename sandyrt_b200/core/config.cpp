@@ -263,6 +263,15 @@ std::map<std::string, Architecture>& table() {
             return describe_pugalix(*g);
         };
         t[pugalix.name] = std::move(pugalix);
+        Architecture migelix;
+        migelix.name = MigelixConfig::kArchitecture;
+        migelix.parse = [](const Json& raw) { return std::unique_ptr<ModelConfig>(new MigelixConfig(MigelixConfig::from_json(raw))); };
+        migelix.describe = [](const ModelConfig& c) {
+            const auto* g = dynamic_cast<const MigelixConfig*>(&c);
+            if (!g) throw ConfigError("Migelix was given another architecture's configuration");
+            return describe_migelix(*g);
+        };
+        t[migelix.name] = std::move(migelix);
     });
     return t;
 }

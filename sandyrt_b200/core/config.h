@@ -197,6 +197,43 @@ public:
     void validate() const override;
 };
 
+// Migelix's config.json (core/migelix.cpp says what the keys mean): layers listed one by one, each time mixing, a windowed
+// attention, or an attention beside a delta rule; a layer may use another's tensors; a dense feed-forward, or none.
+class MigelixConfig : public ModelConfig {
+public:
+    static constexpr const char* kArchitecture = "Migelix";
+    struct Attention {
+        int64_t heads = 0, kv_heads = 0, dim = 0, vdim = 0;
+        double scale = 1.0, softcap = 0.0;                  // softcap 0: none
+        int64_t window = 0;                                 // 0: none
+        int64_t rot_dims = 0;                               // 0: no rotary positions
+        double rot_base = 10000.0;
+        bool yarn = false;
+        double yarn_factor = 1.0, yarn_original = 1.0, yarn_fast = 1.0, yarn_slow = 1.0;
+    };
+    struct Layer {
+        std::string type;                                   // "attention" | "parallel" | "wkv"
+        Attention attention;                                // attention; parallel's left side
+        double left_scale = 1.0, right_scale = 1.0;         // parallel
+        int64_t heads = 0, dim = 0;                         // wkv; parallel's right side
+        int64_t kv_heads = 0, vdim = 0, conv = 0;           // parallel's right side
+        int64_t rank = 0, gate_rank = 0;                    // 0: the weight file's
+        int64_t ff = 0;                                     // 0: the layer has no feed-forward
+        int64_t weights_of = -1;                            // >= 0: the layer whose tensors this one uses
+    };
+    int64_t vocab = 0, width = 0;
+    double norm_eps = 1e-6, logit_softcap = 0.0;            // logit_softcap 0: none
+    std::vector<Layer> layers;
+
+    static MigelixConfig from_json(const Json& raw);
+    std::string architecture() const override { return kArchitecture; }
+    Json to_json() const override;
+    void validate() const override;
+    size_t owner(size_t i) const;                           // the layer whose tensors layer i uses
+private:
+    static Json layer_json(const Layer& l);                 // without weights_of
+};
+
 // A configuration of an architecture defined outside this library: its normalised config.json
 // as the architecture's own `parse` returned it.
 class ForeignConfig : public ModelConfig {
@@ -235,5 +272,6 @@ ModelSpec describe_sovezen(const SovezenConfig& cfg);
 ModelSpec describe_bilurax(const BiluraxConfig& cfg);
 ModelSpec describe_tifepel(const TifepelConfig& cfg);
 ModelSpec describe_pugalix(const PugalixConfig& cfg);
+ModelSpec describe_migelix(const MigelixConfig& cfg);
 
 }  // namespace sandy

@@ -362,6 +362,23 @@ void gemm_skinny(const Launch& l, const Tensor* a, const FusedNorm* norm, const 
     if (kv) kv->written = true;
 }
 
+bool skinny_groups_supported(int64_t M, int64_t N, int64_t K) { return M <= kSkinnyMaxRows && N % 16 == 0 && K % 8 == 0 && K >= 8; }
+
+void gemm_skinny_groups(const Launch& l, const Tensor& a, const Tensor& w, int n_groups, Tensor& out) {
+    const int64_t M = a.rows, K = w.cols, N = n_groups > 0 ? w.rows / n_groups : 0;
+    if (a.dtype != DType::BF16 || w.dtype != DType::BF16) throw UnsupportedShape("gemm_skinny_groups takes bfloat16 operands");
+    if (n_groups <= 0 || w.rows % n_groups || a.cols != n_groups * K || out.rows != M || out.cols != w.rows)
+        throw KernelError("gemm_skinny_groups: shapes disagree: a " + dims(a) + ", w " + dims(w) + ", out " + dims(out));
+    if (!skinny_groups_supported(M, N, K) || w.ld % 8 || a.ld % 8 || ((uintptr_t)w.data & 15) || ((uintptr_t)a.data & 15))
+        throw UnsupportedShape("gemm_skinny_groups: up to 64 rows, K and pitches multiples of 8, N a multiple of 16, operands 16-byte aligned");
+    if (left_out("product", w.rows, K)) return;
+    static auto fn = SANDY_KERNEL(gemm_skinny, sandy_gemm_skinny_groups);
+    OpTimer timer(l, "product, streaming", tensor_bytes(&a) + tensor_bytes(&w) + tensor_bytes(&out), 2.0 * M * w.rows * K);
+    check(fn(a.data, w.data, out.data, (int)M, n_groups, (int)N, (int)K, (int)a.ld, (int)w.ld, (int)out.ld, code_of(out.dtype), l.stream),
+          "gemm_skinny_groups(M=" + std::to_string(M) + ",groups=" + std::to_string(n_groups) + ",N=" + std::to_string(N) +
+              ",K=" + std::to_string(K) + ")");
+}
+
 // ---- 17 to 64 rows on the tensor cores -----------------------------------------------------------------
 // Which kernel a product of 17 to 64 rows gets.  Timed one kernel after itself the tcgen05 kernel with
 // 64-wide tiles wins the up-projection (3072 x 768 at 64 rows: 6.8 us against 9.8 streaming) and split-K
@@ -626,16 +643,16 @@ void rmsnorm(const Launch& l, const Tensor& x, const Tensor* gain, float eps, Te
 void rmsnorm_shift(const Launch& l, const StepSeqs& s, const Tensor& x, const Tensor* gain, float eps, const Tensor& mix,
                    const StateView& state, Tensor& out, int max_q_len) {
     if (x.dtype != DType::F32 || (gain && (gain->dtype != DType::F32 || gain->numel() != x.cols)) || mix.dtype != DType::F32 ||
-        mix.numel() != x.cols || out.rows != x.rows || out.cols != x.cols || state.dtype != DType::F32 || state.row_elems < x.cols ||
+        x.cols == 0 || mix.numel() % x.cols || !mix.contiguous() || out.rows != x.rows || out.cols != mix.numel() || state.dtype != DType::F32 || state.row_elems < x.cols ||
         x.rows != s.n_tokens)
-        throw KernelError("rmsnorm_shift: float32 x [T, width], gain and mix [width], a float32 state of at least width floats expected");
+        throw KernelError("rmsnorm_shift: float32 x [T, width], gain [width], mix [n, width], out [T, n * width] and a float32 state of at least width floats expected");
     if (left_out("layernorm")) return;
-    static auto fn = SANDY_KERNEL(rmsnorm, sandy_rmsnorm_shift);
+    static auto fn = SANDY_KERNEL(rmsnorm, sandy_rmsnorm_shifts);
     static auto keep = SANDY_KERNEL(rmsnorm, sandy_rmsnorm_keep);
     const float* g = gain ? (const float*)gain->data : nullptr;
     {
-        OpTimer timer(l, "rmsnorm + token shift", (double)x.rows * x.cols * (2 * x.elem_size() + out.elem_size()), 0);
-        check(fn((const float*)x.data, (int)x.ld, g, (const float*)mix.data, (float*)state.data, (long long)state.row_elems,
+        OpTimer timer(l, "rmsnorm + token shift", (double)x.rows * x.cols * 2 * x.elem_size() + tensor_bytes(&out), 0);
+        check(fn((const float*)x.data, (int)x.ld, g, (const float*)mix.data, (int)(mix.numel() / x.cols), (float*)state.data, (long long)state.row_elems,
                  s.token_seq, s.q_start, s.seq_slots, out.data, (int)out.ld, s.n_tokens, (int)x.cols, eps, code_of(out.dtype), l.stream),
               "rmsnorm_shift(width=" + std::to_string(x.cols) + ")");
     }
@@ -896,7 +913,7 @@ void attention_prepare(const Launch& l, const AttentionPrepare& p, const Tensor&
              c.head_dim, p.q_gain, p.k_gain, p.eps, p.freq, p.rot_dims, positions, token_seq, block_table, max_blocks, c.k, c.v,
              c.page_stride, c.page_size, c.num_pages, p.write_cache ? 1 : 0, q_out.data, (int)q_out.ld, p.gate_in, p.ld_gate,
              p.gate_out, p.gate_scale, p.q_head_scale, p.v_unit_eps, p.per_head_norm ? 1 : 0, p.q_pos_coef, p.q_pos_every,
-             p.interleaved ? 1 : 0, code_of(proj.dtype), l.kernel_status, l.stream),
+             p.interleaved ? 1 : 0, p.rot_scale, code_of(proj.dtype), l.kernel_status, l.stream),
           "attention_prepare");
 }
 
@@ -907,18 +924,21 @@ int64_t mlstm_state_floats(int n_heads, int qk_dim, int v_dim) {
 }
 
 void delta_prepare(const Launch& l, const StepSeqs& s, const DeltaShape& d, const Tensor& proj, const Tensor& taps,
-                   const Tensor& gates, const float* a_log, const float* dt_bias, const StateView& state, int64_t tail_off,
-                   float q_scale, Tensor& qkv, Tensor& bg) {
+                   const Tensor* gates, const float* a_log, const float* dt_bias, const StateView& state, int64_t tail_off,
+                   float q_scale, Tensor& qkv, Tensor* bg, int max_q_len) {
     const int64_t channels = 2 * (int64_t)d.n_qk_heads * d.qk_dim + (int64_t)d.n_heads * d.v_dim;
-    if (proj.cols < channels || taps.dtype != DType::F32 || taps.numel() != channels * d.n_taps || gates.dtype != DType::F32 ||
-        gates.cols < 2 * d.n_heads || qkv.dtype != DType::F32 || qkv.cols != channels || bg.dtype != DType::F32 ||
-        bg.cols != 2 * d.n_heads || !bg.contiguous() || state.dtype != DType::F32)
+    if (proj.cols < channels || taps.dtype != DType::F32 || taps.numel() != channels * d.n_taps || (gates != nullptr) != (bg != nullptr) ||
+        (gates && (gates->dtype != DType::F32 || gates->cols < 2 * d.n_heads || bg->dtype != DType::F32 || bg->cols != 2 * d.n_heads ||
+                   !bg->contiguous())) ||
+        qkv.dtype != DType::F32 || qkv.cols != channels || state.dtype != DType::F32 ||
+        tail_off + (int64_t)(d.n_taps - 1) * channels > state.row_elems)
         throw KernelError("delta_prepare: shapes disagree");
-    static auto fn = SANDY_KERNEL(matrix_state, sandy_delta_prepare);
+    static auto fn = SANDY_KERNEL(matrix_state, sandy_delta_prepare_keep);
     OpTimer timer(l, "delta rule: conv + norms + gates", tensor_bytes(&proj) + tensor_bytes(&qkv), 0);
-    check(fn(proj.data, (int)proj.ld, code_of(proj.dtype), (const float*)taps.data, d.n_taps, (const float*)gates.data, (int)gates.ld,
-             a_log, dt_bias, (const float*)state.data, state.row_elems, tail_off, s.token_seq, s.q_start, s.seq_slots,
-             (float*)qkv.data, (int)qkv.ld, (float*)bg.data, s.n_tokens, d.n_heads, d.n_qk_heads, d.qk_dim, d.v_dim, q_scale, l.stream),
+    check(fn(proj.data, (int)proj.ld, code_of(proj.dtype), (const float*)taps.data, d.n_taps, gates ? (const float*)gates->data : nullptr,
+             gates ? (int)gates->ld : 0, a_log, dt_bias, (float*)state.data, state.row_elems, tail_off, s.token_seq, s.q_start, s.seq_slots,
+             (float*)qkv.data, (int)qkv.ld, bg ? (float*)bg->data : nullptr, s.n_tokens, d.n_heads, d.n_qk_heads, d.qk_dim, d.v_dim, q_scale,
+             max_q_len == 1 ? 1 : 0, l.stream),
           "delta_prepare");
 }
 
@@ -1112,34 +1132,47 @@ void mlstm_scan(const Launch& l, const StepSeqs& s, const MlstmShape& m, const T
               "mlstm_chunk_scan" + shape);
 }
 
-int64_t gla_state_floats(const GlaShape& m) { return (int64_t)m.n_heads * m.v_dim * m.qk_dim; }
+int64_t fade_state_floats(const FadeShape& m) { return (int64_t)m.n_heads * m.v_dim * m.qk_dim; }
 
-void gla_scan(const Launch& l, const StepSeqs& s, const GlaShape& m, const Tensor& proj, const Tensor& low, const Tensor& w2t,
-              const Tensor& bias, const StateView& state, Tensor& out, int max_q_len, Workspace& ws) {
+void fade_scan(const Launch& l, const StepSeqs& s, const FadeShape& m, const Tensor& proj, const Tensor& low, const Tensor& w2t,
+               const Tensor& bias, const StateView& state, Tensor& out, int max_q_len, Workspace& ws) {
     const int64_t HD = (int64_t)m.n_heads * m.qk_dim;
     if (out.dtype != DType::F32 || out.cols != (int64_t)m.n_heads * m.v_dim || low.dtype != DType::F32 || w2t.dtype != DType::F32 ||
         w2t.rows != low.cols || w2t.cols != HD || !w2t.contiguous() || bias.dtype != DType::F32 || bias.numel() != HD ||
-        state.dtype != DType::F32 || state.row_elems < gla_state_floats(m) || proj.rows != s.n_tokens || low.rows != s.n_tokens)
-        throw KernelError("gla_scan: shapes disagree");
-    static auto fn = SANDY_KERNEL(gated_linear, sandy_gla_scan);
-    static auto chunked = SANDY_KERNEL(gated_linear, sandy_gla_chunk_scan);
-    static auto need = SANDY_KERNEL(gated_linear, sandy_gla_scratch_floats);
+        state.dtype != DType::F32 || m.state_off < 0 || state.row_elems < m.state_off + fade_state_floats(m) || proj.rows != s.n_tokens ||
+        low.rows != s.n_tokens ||
+        (m.beta && (m.beta->dtype != DType::F32 || m.beta->cols < m.n_heads || m.beta->rows != s.n_tokens)))
+        throw KernelError("fade_scan: shapes disagree");
+    static auto fn = SANDY_KERNEL(gated_linear, sandy_fade_scan);
+    static auto chunked = SANDY_KERNEL(gated_linear, sandy_fade_chunk_scan);
+    static auto need = SANDY_KERNEL(gated_linear, sandy_fade_scratch_floats);
+    SandyFadeRule rule = {};
+    rule.kind = (int)m.kind;
+    rule.decay = (int)m.decay;
+    rule.inv_tau = m.inv_tau;
+    rule.tanh_low = m.tanh_low ? 1 : 0;
+    rule.a_log = m.a_log;
+    rule.bonus = m.bonus;
+    rule.beta = m.beta ? (const float*)m.beta->data : nullptr;
+    rule.ld_beta = m.beta ? (int)m.beta->ld : 0;
+    rule.n_qk_heads = m.n_qk_heads;
+    static const char* const names[] = {"gated linear attention: recurrence", "time mixing: recurrence", "delta rule by channel: recurrence"};
     const int long_from = max_q_len >= kChunkedFrom ? kChunkedFrom : 0;
     const double st = 2.0 * s.n_seqs * m.n_heads * m.qk_dim * m.v_dim * 4.0;
     const std::string shape = "(d=" + std::to_string(m.qk_dim) + ",e=" + std::to_string(m.v_dim) + ")";
-    float* scratch = long_from ? (float*)ws.raw("gla_chunks", (size_t)need(s.n_tokens, s.n_seqs, m.n_heads, m.qk_dim) * sizeof(float)) : nullptr;
-    OpTimer timer(l, "gated linear attention: recurrence", st + tensor_bytes(&out), 4.0 * s.n_tokens * m.n_heads * m.qk_dim * m.v_dim);
+    float* S = (float*)state.data + m.state_off;
+    float* scratch = long_from ? (float*)ws.raw("fade_chunks", (size_t)need(rule.kind, s.n_tokens, s.n_seqs, m.n_heads, m.qk_dim, m.v_dim) * sizeof(float)) : nullptr;
+    OpTimer timer(l, names[(int)m.kind], st + tensor_bytes(&out), (m.kind == FadeKind::Delta ? 6.0 : 4.0) * s.n_tokens * m.n_heads * m.qk_dim * m.v_dim);
     check(fn(proj.data, (int)proj.ld, code_of(proj.dtype), m.q_off, m.k_off, m.v_off, (const float*)low.data, (int)low.ld, (int)low.cols,
-             (const float*)w2t.data, (const float*)bias.data, m.inv_tau, m.q_scale, (float*)state.data, state.row_elems, s.q_start,
-             s.seq_slots, (float*)out.data, (int)out.ld, s.n_seqs, m.n_heads, m.qk_dim, m.v_dim, long_from, l.stream),
-          "gla_scan" + shape);
+             (const float*)w2t.data, (const float*)bias.data, &rule, m.q_scale, S, state.row_elems, s.q_start, s.seq_slots,
+             (float*)out.data, (int)out.ld, s.n_seqs, m.n_heads, m.qk_dim, m.v_dim, long_from, l.stream),
+          "fade_scan" + shape);
     if (!long_from) return;
     g_launches++;                                          // two launches
     check(chunked(proj.data, (int)proj.ld, code_of(proj.dtype), m.q_off, m.k_off, m.v_off, (const float*)low.data, (int)low.ld, (int)low.cols,
-                  (const float*)w2t.data, (const float*)bias.data, m.inv_tau, m.q_scale, (float*)state.data, state.row_elems, s.q_start,
-                  s.seq_slots, (float*)out.data, (int)out.ld, scratch, s.n_tokens, s.n_seqs, max_q_len, m.n_heads, m.qk_dim, m.v_dim,
-                  long_from, l.stream),
-          "gla_chunk_scan" + shape);
+                  (const float*)w2t.data, (const float*)bias.data, &rule, m.q_scale, S, state.row_elems, s.q_start, s.seq_slots,
+                  (float*)out.data, (int)out.ld, scratch, s.n_tokens, s.n_seqs, max_q_len, m.n_heads, m.qk_dim, m.v_dim, long_from, l.stream),
+          "fade_chunk_scan" + shape);
 }
 
 void sample(const Launch& l, const Tensor& logits, int* out_tokens, const float* temperature, const int* top_k,

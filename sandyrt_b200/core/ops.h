@@ -12,6 +12,7 @@
 #include <string>
 #include <vector>
 
+#include "../csrc/gated_linear.h"
 #include "../csrc/matrix_state.h"
 #include "cache.h"
 #include "device.h"
@@ -97,6 +98,10 @@ constexpr int kSkinnyNormPaysK = 1024;
 void gemm_skinny(const Launch& l, const Tensor* a, const FusedNorm* norm, const Tensor& w, const Tensor* bias, Tensor& out,
                  Act act, const Tensor* residual, KVTarget* kv = nullptr);
 constexpr int kSkinnyMaxRows = 64;
+// n_groups products of one shape in one launch: w [n_groups * N, K], a [M, n_groups * K], out [M, n_groups * N]; columns g of out
+// are columns g of a times rows g of w.  Up to kSkinnyMaxRows rows, N a multiple of 16.
+bool skinny_groups_supported(int64_t M, int64_t N, int64_t K);
+void gemm_skinny_groups(const Launch& l, const Tensor& a, const Tensor& w, int n_groups, Tensor& out);
 // tcgen05 with the weight as the wide operand and K split over a cluster, for 17 to 64 rows (gemm_small.cu).
 // small_gemm_kernel: which kernel a bfloat16 product of 17 to 64 rows gets, from its shape alone.
 // The split-K kernel also takes 65 to 256 rows (a short prompt step, or a portion of one): products with a
@@ -173,7 +178,8 @@ void rmsnorm(const Launch& l, const Tensor& x, const Tensor* gain, float eps, Te
 // Token shift behind the norm: h[t] = norm(x[t]) * gain, out[t] = h[t] + (h[t-1] - h[t]) * mix, where the h before a
 // request's first token of the step is the first x.cols floats of its state row (zeros at a request's very first
 // token: a slot is cleared on admission), and the row then takes the h of the request's last token.  All 32-bit; out
-// in its own type.  `max_q_len` is the step's longest portion (one launch when it is 1, two otherwise).
+// in its own type.  `max_q_len` is the step's longest portion (one launch when it is 1, two otherwise).  mix may have several
+// rows ([n, x.cols]): out is then [T, n * x.cols], the results side by side.
 void rmsnorm_shift(const Launch& l, const StepSeqs& s, const Tensor& x, const Tensor* gain, float eps, const Tensor& mix,
                    const StateView& state, Tensor& out, int max_q_len);
 // x += mult * y / sqrt(mean(y^2) + eps) * gain; both float32.
@@ -276,7 +282,8 @@ struct AttentionPrepare {
     float eps = 0.0f;
     const float* freq = nullptr;                                   // rotary frequencies [rot_dims / 2], or null
     int rot_dims = 0;
-    const float* gate_in = nullptr;                                // float32 [T, ld_gate]: per-head gate pre-activations
+    const float* gate_in = nullptr;                                // float32 [T, ld_gate]: per-head gate pre-activations; null with
+                                                                   // gate_out: gate_scale alone
     int ld_gate = 0;
     float* gate_out = nullptr;                                     // float32 [T, H]: sigmoid(gate_in) * gate_scale
     float gate_scale = 1.0f;
@@ -287,6 +294,7 @@ struct AttentionPrepare {
     float q_pos_coef = 0.0f;                                       // with q_pos_every > 0 the query at position p is multiplied by
     int q_pos_every = 0;                                           // 1 + q_pos_coef * ln(floor((p + 1) / q_pos_every) + 1)
     bool interleaved = false;                                      // the rotation pairs 2i with 2i + 1 (else i with i + rot_dims / 2)
+    float rot_scale = 1.0f;                                        // a factor on the rotation's cosine and sine
     bool write_cache = true;
 };
 void attention_prepare(const Launch& l, const AttentionPrepare& p, const Tensor& proj, const KVView& cache,
@@ -299,10 +307,11 @@ int64_t mlstm_state_floats(int n_heads, int qk_dim, int v_dim);
 struct DeltaShape { int n_heads = 0, n_qk_heads = 0, qk_dim = 0, v_dim = 0, n_taps = 0; };
 // conv + silu + unit vectors + gates.  proj [T, >= channels] (q, k, v channels first); taps float32 [channels, n_taps];
 // gates float32 [T, 2H] (beta's pre-activation, then the decay's); qkv float32 [T, channels]; bg float32 [T, 2H]
-// (beta, then the logarithm of the decay).
+// (beta, then the logarithm of the decay).  `gates` and `bg` null: no gates are formed.  With `max_q_len` 1 (every request brings
+// one token) the convolution's tail moves on in the same launch; conv_tail does it otherwise (0: always).
 void delta_prepare(const Launch& l, const StepSeqs& s, const DeltaShape& d, const Tensor& proj, const Tensor& taps,
-                   const Tensor& gates, const float* a_log, const float* dt_bias, const StateView& state, int64_t tail_off,
-                   float q_scale, Tensor& qkv, Tensor& bg);
+                   const Tensor* gates, const float* a_log, const float* dt_bias, const StateView& state, int64_t tail_off,
+                   float q_scale, Tensor& qkv, Tensor* bg, int max_q_len = 0);
 void conv_tail(const Launch& l, const StepSeqs& s, const DeltaShape& d, const Tensor& proj, const StateView& state,
                int64_t tail_off);
 // From how many tokens of one request on a step's recurrence runs a chunk of tokens at a time (parallel inside the
@@ -318,16 +327,30 @@ struct MlstmShape { int n_heads = 0, qk_dim = 0, v_dim = 0, q_off = 0, k_off = 0
 void mlstm_scan(const Launch& l, const StepSeqs& s, const MlstmShape& m, const Tensor& proj, const Tensor& gates,
                 const float* gate_bias, const StateView& state, Tensor& out, int max_q_len);
 
-// ---- gated linear attention: a decay per key channel and token (gated_linear.cu) --------------------------------
-struct GlaShape {
-    int n_heads = 0, qk_dim = 0, v_dim = 0, q_off = 0, k_off = 0, v_off = 0;      // columns of q, k, v in the projection
-    float inv_tau = 1.0f, q_scale = 1.0f;
+// ---- recurrences with a decay per key channel and token (gated_linear.cu) ----------------------------------------
+enum class FadeKind : int { Add = SANDY_FADE_ADD, Bonus = SANDY_FADE_BONUS, Delta = SANDY_FADE_DELTA };
+enum class DecayForm : int { LogSigmoid = SANDY_DECAY_LOGSIGMOID, Exp = SANDY_DECAY_EXP, Softplus = SANDY_DECAY_SOFTPLUS };
+struct FadeShape {
+    int n_heads = 0, n_qk_heads = 0;                               // n_qk_heads 0: as many as heads
+    int qk_dim = 0, v_dim = 0, q_off = 0, k_off = 0, v_off = 0;    // columns of q, k, v in the projection
+    float q_scale = 1.0f;
+    FadeKind kind = FadeKind::Add;
+    DecayForm decay = DecayForm::LogSigmoid;
+    float inv_tau = 1.0f;                                          // LogSigmoid
+    bool tanh_low = false;
+    const float* a_log = nullptr;                                  // float32 [H], Softplus
+    const float* bonus = nullptr;                                  // float32 [H * qk_dim], Bonus
+    const Tensor* beta = nullptr;                                  // float32 [T, H]: pre-activations of the step size, Delta
+    int64_t state_off = 0;                                         // where S begins in a request's state
 };
-int64_t gla_state_floats(const GlaShape& m);                       // S [H][v_dim][qk_dim]
-// S_t = diag(alpha_t) S_(t-1) + k_t v_t^T, out_t = S_t^T (q_t q_scale); alpha = sigmoid(low w2t + bias)^inv_tau per key channel.
+int64_t fade_state_floats(const FadeShape& m);                     // S [H][v_dim][qk_dim]
+// With z = w2 low + bias (or w2 tanh(low) + bias) per head and key channel and D_t = diag of the decays that follow from it:
+//   Add     S_t = D_t S_(t-1) + k_t v_t^T,                     out_t = S_t^T (q_t q_scale)
+//   Bonus   the same state,                                    out_t = (S_(t-1) + diag(bonus) k_t v_t^T)^T (q_t q_scale)
+//   Delta   S' = D_t S_(t-1), S_t = S' + k_t u_t^T with u_t = sigmoid(beta_t) (v_t - S'^T k_t),   out_t = S_t^T (q_t q_scale)
 // low float32 [T, rank]; w2t float32 [rank, H * qk_dim]; bias float32 [H * qk_dim]; out float32 [T, H * v_dim].
-void gla_scan(const Launch& l, const StepSeqs& s, const GlaShape& m, const Tensor& proj, const Tensor& low, const Tensor& w2t,
-              const Tensor& bias, const StateView& state, Tensor& out, int max_q_len, Workspace& ws);
+void fade_scan(const Launch& l, const StepSeqs& s, const FadeShape& m, const Tensor& proj, const Tensor& low, const Tensor& w2t,
+               const Tensor& bias, const StateView& state, Tensor& out, int max_q_len, Workspace& ws);
 
 // The last n_taps - 1 rows of `rows` ([T, channels], any pitch) of every request into its state at tail_off, as the
 // convolutions above keep theirs (rows before the step come from the old tail).

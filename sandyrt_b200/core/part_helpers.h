@@ -24,6 +24,9 @@ TensorRequest want(std::vector<int64_t> shape, const char* init = "weight");
 int64_t round_up(int64_t n, int64_t m);
 // f_i = base^(-2i / dims), i < dims / 2, with an optional long-context rescaling {factor, low, high, original}.
 std::vector<float> rotary_frequencies(int dims, double base, const Json* scaling);
+// The same under YaRN's rescaling {factor, original, fast, slow}: see parts_hybrid.cpp.  `magnitude` is its factor on the
+// rotation's cosine and sine.
+std::vector<float> yarn_frequencies(int dims, double base, const Json& scaling, float& magnitude);
 DeviceWeight floats_to_device(const std::vector<float>& v);
 
 }  // namespace part_helpers

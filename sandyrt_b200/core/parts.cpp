@@ -126,6 +126,23 @@ void Linear::run(StepContext& ctx, NormedInput* lazy, const Tensor* a, Tensor& o
     }
 }
 
+void Linear::run_groups(StepContext& ctx, const Tensor& a, int n_groups, Tensor& out) {
+    if (has_bias_ || !w_out_in_ || n_groups <= 0 || out_ % n_groups || a.cols != n_groups * in_)
+        throw KernelError("Linear " + name_ + ": groups want stacked [out, in] weights without a bias, and an input as wide as all of them");
+    const int64_t N = out_ / n_groups;
+    if (use_tc_ && ops::skinny_groups_supported(a.rows, N, in_)) {
+        ops::gemm_skinny_groups(ctx.launch, a, weight_.view, n_groups, out);
+        return;
+    }
+    for (int g = 0; g < n_groups; g++) {
+        const Tensor ag = a.col_range(g * in_, (g + 1) * in_), wg = weight_.view.row_range(g * N, (g + 1) * N);
+        Tensor og = out.col_range(g * N, (g + 1) * N);
+        if (use_tc_ && a.rows <= ops::kSkinnyMaxRows) ops::gemm_skinny(ctx.launch, &ag, nullptr, wg, nullptr, og, ops::Act::None, nullptr);
+        else if (use_tc_) ops::gemm_tc(ctx.launch, ag, wg, nullptr, og, ops::Act::None, nullptr);
+        else ops::gemm_simt(ctx.launch, ag, wg, nullptr, og, true, ops::Act::None, nullptr);
+    }
+}
+
 // ---- built-in parts -----------------------------------------------------------------------------------------
 namespace {
 

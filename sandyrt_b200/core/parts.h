@@ -254,6 +254,9 @@ public:
     // kernel used can write keys/values into the cache, it does and sets kv->written.
     void run(StepContext& ctx, NormedInput* lazy, const Tensor* a, Tensor& out, ops::Act act, const Tensor* residual,
              ops::KVTarget* kv = nullptr);
+    // Several products of one shape whose weights are stacked in this one ([n_groups * N, in], layout "out_in", no bias): columns
+    // g of out [T, n_groups * N] = columns g of a [T, n_groups * in] times rows g.  Up to 64 rows they are one launch.
+    void run_groups(StepContext& ctx, const Tensor& a, int n_groups, Tensor& out);
     const Tensor& weight() const { return weight_.view; }
 private:
     int64_t in_, out_;
@@ -296,8 +299,9 @@ void register_latent_parts();
 // with a learned bias by distance, and the state-space mixer with one decay per head.
 void register_stream_parts();
 
-// Kinds of parts_linear.cpp: attention with a sliding window that keeps the first tokens, a one in the softmax's
-// denominator and a gate by element; gated linear attention; the matrix memory as a mixer of its own.
+// Kinds of parts_linear.cpp: attention with a sliding window that keeps the first tokens, a sink in the softmax's denominator
+// and a gate by element; gated linear attention; the matrix memory as a mixer of its own; the delta rule with a decay per key
+// channel, alone and beside attention; time mixing.
 void register_linear_parts();
 
 template <typename T>

@@ -104,6 +104,24 @@ std::vector<float> rotary_frequencies(int dims, double base, const Json* scaling
     return out;
 }
 
+// YaRN: a pair of entries that turns at least `fast` times within the original length keeps its frequency, one that turns at
+// most `slow` times is slowed down by factor, and between the two the share of the slow one grows linearly with the pair's index.
+// The entry whose wavelength fits t times into the original length is dims ln(original / (2 pi t)) / (2 ln base).
+std::vector<float> yarn_frequencies(int dims, double base, const Json& scaling, float& magnitude) {
+    const double factor = scaling.at("factor").as_double(), original = scaling.at("original").as_double();
+    auto entry = [&](double turns) { return dims * std::log(original / (2.0 * kPi * turns)) / (2.0 * std::log(base)); };
+    const double lo = std::max(std::floor(entry(scaling.at("fast").as_double())), 0.0);
+    const double hi = std::min(std::ceil(entry(scaling.at("slow").as_double())), (double)(dims - 1));
+    std::vector<float> out;
+    for (int i = 0; i < dims / 2; i++) {
+        const double f = std::pow(base, -2.0 * i / dims);
+        const double slowed = std::min(std::max((i - lo) / std::max(hi - lo, 0.001), 0.0), 1.0);
+        out.push_back((float)(f / factor * slowed + f * (1.0 - slowed)));
+    }
+    magnitude = (float)(0.1 * std::log(factor) + 1.0);
+    return out;
+}
+
 DeviceWeight floats_to_device(const std::vector<float>& v) {
     auto buf = alloc_f32(v.size());
     std::copy(v.begin(), v.end(), buf.get());
@@ -116,12 +134,22 @@ namespace {
 using namespace part_helpers;
 
 // ---- RMS norm --------------------------------------------------------------------------------------------
-// Parameters: width, eps.  Tensor: "weight" (a plain gain, not one-plus).
+// Parameters: width, eps, gain_offset (absent: 0).  Tensor: "weight"; the gain is gain_offset + weight, formed in 32-bit (an
+// offset of 1: weights stored around zero).
 class RMSNorm : public Norm {
 public:
-    explicit RMSNorm(const PartSpec& s) : Norm(s), width_(s.get_int("width")), eps_((float)s.get_double("eps")) {}
-    TensorRequests requests() const override { return {{"weight", want({width_}, "gamma")}}; }
-    void bind(const TensorMap& t, DType) override { gain_ = to_device(t.at("weight"), DType::F32); }
+    explicit RMSNorm(const PartSpec& s)
+        : Norm(s), width_(s.get_int("width")), eps_((float)s.get_double("eps")), offset_((float)s.get_double("gain_offset", 0.0)) {}
+    TensorRequests requests() const override { return {{"weight", want({width_}, offset_ == 0.0f ? "gamma" : "beta")}}; }
+    void bind(const TensorMap& t, DType) override {
+        if (offset_ == 0.0f) {
+            gain_ = to_device(t.at("weight"), DType::F32);
+            return;
+        }
+        std::vector<float> g = to_f32(t.at("weight"));
+        for (float& v : g) v += offset_;
+        gain_ = floats_to_device(g);
+    }
     size_t weight_bytes() const override { return gain_.bytes(); }
     void forward(StepContext& ctx, const Tensor& x, Tensor& out, const int* rows, int n_rows) override {
         ops::rmsnorm(ctx.launch, x, &gain_.view, eps_, out, rows, n_rows);
@@ -136,7 +164,7 @@ public:
     }
 private:
     int64_t width_;
-    float eps_;
+    float eps_, offset_;
     DeviceWeight gain_;
 };
 
@@ -478,9 +506,9 @@ public:
         ops::DeltaShape ds{H_, G_, d_, e_, taps_};
         Tensor qkv = ws.get("delta_qkv", T, channels_, DType::F32);
         Tensor bg = ws.get("delta_gates", T, 2 * H_, DType::F32);
-        ops::delta_prepare(l, seqs, ds, wide, conv_.view, gates, (const float*)a_log_.view.data, (const float*)dt_bias_.view.data,
-                           state, tail_off, 1.0f / std::sqrt((float)d_), qkv, bg);
-        ops::conv_tail(l, seqs, ds, wide, state, tail_off);
+        ops::delta_prepare(l, seqs, ds, wide, conv_.view, &gates, (const float*)a_log_.view.data, (const float*)dt_bias_.view.data,
+                           state, tail_off, 1.0f / std::sqrt((float)d_), qkv, &bg, ctx.max_q_len);
+        if (ctx.max_q_len != 1) ops::conv_tail(l, seqs, ds, wide, state, tail_off);
         Tensor read = ws.get("mix_read", T, (int64_t)H_ * e_, DType::F32);
         ops::delta_scan(l, seqs, ds, qkv, bg, state, read, ctx.max_q_len);
         Tensor normed = ws.get("delta_normed", T, (int64_t)H_ * e_, ctx.compute_dtype);

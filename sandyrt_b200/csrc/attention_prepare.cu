@@ -5,15 +5,17 @@
 //   2. optional rotary position encoding of queries and keys on the first `rot_dims` entries of every head
 //      ("rotate half": entry i pairs with entry i + rot_dims / 2; or interleaved: 2i with 2i + 1; the pair (u, v) at position p becomes
 //      (u cos a - v sin a, v cos a + u sin a), a = p * freq[i]), positions and angles in 32-bit; the
-//      frequencies come from the caller, who has applied whatever rescaling the model wants;
+//      frequencies come from the caller, who has applied whatever rescaling the model wants, and so does a factor on
+//      cosine and sine;
 //   3. keys and values written into the request's pages, queries into a dense matrix, each head padded
 //      with zeros from its own size up to the cache's head size (key size and value size may differ: the
 //      cache and the attention kernels see one head size, the larger of the two rounded up to 16);
 //      optionally each query head times a number of its own (a learned temperature: it reaches the scores through
 //      the query), and each value head divided by its root mean square over its own entries (eps inside the root,
-//      no gain), in 32-bit, so that the cache holds unit-RMS values;
+//      no gain), in 32-bit, so that the cache holds unit-RMS values.  Where values are keys (as projected, before they
+//      turn), v_off is k_off;
 //   4. optional per-head output gate: gate_out[t, h] = sigmoid(gate_in[t, h]) * gate_scale, 32-bit, which
-//      the attention kernels multiply into a head's output.
+//      the attention kernels multiply into a head's output; gate_scale alone where there is no gate_in.
 //
 // One block per token.  The step's tokens find their pages as everywhere: token -> request -> block table.
 #include "common.cuh"
@@ -33,7 +35,7 @@ attention_prepare_kernel(const T* __restrict__ proj, int ld, int q_off, int k_of
                          T* __restrict__ q_out, int ld_q, const float* __restrict__ gate_in, int ld_gate,
                          float* __restrict__ gate_out, float gate_scale, const float* __restrict__ q_head_scale,
                          float v_unit_eps, int per_head_norm, float q_pos_coef, int q_pos_every, int interleaved,
-                         int* __restrict__ status) {
+                         float rot_scale, int* __restrict__ status) {
     __shared__ float scratch[32];
     extern __shared__ float cs[];                    // cos [rot_dims / 2], sin [rot_dims / 2], then 1 / rms of each value head,
     float* v_inv = cs + rot_dims;                    // then (per_head_norm) 1 / rms of each query head and each key head
@@ -46,8 +48,8 @@ attention_prepare_kernel(const T* __restrict__ proj, int ld, int q_off, int k_of
             const float a = (float)pos * freq[i];
             float s, c;
             sincosf(a, &s, &c);
-            cs[i] = c;
-            cs[half + i] = s;
+            cs[i] = c * rot_scale;
+            cs[half + i] = s * rot_scale;
         }
     pdl_wait();
     pdl_launch_dependents();
@@ -139,7 +141,7 @@ attention_prepare_kernel(const T* __restrict__ proj, int ld, int q_off, int k_of
     (void)nv;
     if (gate_out)
         for (int h = threadIdx.x; h < n_heads; h += blockDim.x)
-            gate_out[(size_t)t * n_heads + h] = gate_scale / (1.0f + expf(-gate_in[(size_t)t * ld_gate + h]));
+            gate_out[(size_t)t * n_heads + h] = gate_in ? gate_scale / (1.0f + expf(-gate_in[(size_t)t * ld_gate + h])) : gate_scale;
 }
 
 }  // namespace
@@ -152,7 +154,8 @@ attention_prepare_kernel(const T* __restrict__ proj, int ld, int q_off, int k_of
 // per_head_norm != 0: every query head and every key head is divided by its own root mean square over qk_dim (eps inside
 // the root; the gains, [heads * qk_dim], may then be null) instead of the norm over the whole row.  q_pos_every > 0: the
 // query at position p is multiplied by 1 + q_pos_coef * ln(floor((p + 1) / q_pos_every) + 1).
-// interleaved != 0: the rotation pairs entries 2i and 2i + 1 instead of i and i + rot_dims / 2.
+// interleaved != 0: the rotation pairs entries 2i and 2i + 1 instead of i and i + rot_dims / 2; rot_scale: a factor on cosine and
+// sine.  gate_out without gate_in: gate_scale for every head.
 SANDY_API int sandy_attention_prepare_rot(const void* proj, int ld, int q_off, int k_off, int v_off, int n_tokens, int n_heads,
                                       int n_kv_heads, int qk_dim, int v_dim, int pad_dim, const float* q_gain,
                                       const float* k_gain, float eps, const float* freq, int rot_dims, const int* positions,
@@ -160,12 +163,12 @@ SANDY_API int sandy_attention_prepare_rot(const void* proj, int ld, int q_off, i
                                       void* v_cache, long long page_stride, int page_size, int num_pages, int write_cache,
                                       void* q_out, int ld_q, const float* gate_in, int ld_gate, float* gate_out,
                                       float gate_scale, const float* q_head_scale, float v_unit_eps, int per_head_norm,
-                                      float q_pos_coef, int q_pos_every, int interleaved, int dtype, int* status,
-                                      cudaStream_t stream) {
+                                      float q_pos_coef, int q_pos_every, int interleaved, float rot_scale, int dtype,
+                                      int* status, cudaStream_t stream) {
     if (n_tokens == 0) return SANDY_OK;
     if (!proj || !positions || !token_seq || !q_out || (write_cache && (!block_table || !k_cache || !v_cache)))
         return SANDY_ERR_ARGUMENT;
-    if (pad_dim < qk_dim || pad_dim < v_dim || rot_dims < 0 || rot_dims > qk_dim || (rot_dims & 1) || (gate_out && !gate_in))
+    if (pad_dim < qk_dim || pad_dim < v_dim || rot_dims < 0 || rot_dims > qk_dim || (rot_dims & 1))
         return SANDY_ERR_UNSUPPORTED;
     const size_t smem = ((size_t)rot_dims + (size_t)n_kv_heads + (per_head_norm ? (size_t)(n_heads + n_kv_heads) : 0)) * sizeof(float);
     if (smem > 32 * 1024) return SANDY_ERR_UNSUPPORTED;
@@ -174,13 +177,13 @@ SANDY_API int sandy_attention_prepare_rot(const void* proj, int ld, int q_off, i
                             ld, q_off, k_off, v_off, n_heads, n_kv_heads, qk_dim, v_dim, pad_dim, q_gain, k_gain, eps, freq,
                             rot_dims, positions, token_seq, block_table, max_blocks, (float*)k_cache, (float*)v_cache,
                             page_stride, page_size, num_pages, write_cache, (float*)q_out, ld_q, gate_in, ld_gate, gate_out,
-                            gate_scale, q_head_scale, v_unit_eps, per_head_norm, q_pos_coef, q_pos_every, interleaved, status);
+                            gate_scale, q_head_scale, v_unit_eps, per_head_norm, q_pos_coef, q_pos_every, interleaved, rot_scale, status);
     if (dtype == SANDY_BF16)
         return sandy_launch(attention_prepare_kernel<bf16>, dim3(n_tokens), dim3(THREADS), smem, stream, (const bf16*)proj,
                             ld, q_off, k_off, v_off, n_heads, n_kv_heads, qk_dim, v_dim, pad_dim, q_gain, k_gain, eps, freq,
                             rot_dims, positions, token_seq, block_table, max_blocks, (bf16*)k_cache, (bf16*)v_cache,
                             page_stride, page_size, num_pages, write_cache, (bf16*)q_out, ld_q, gate_in, ld_gate, gate_out,
-                            gate_scale, q_head_scale, v_unit_eps, per_head_norm, q_pos_coef, q_pos_every, interleaved, status);
+                            gate_scale, q_head_scale, v_unit_eps, per_head_norm, q_pos_coef, q_pos_every, interleaved, rot_scale, status);
     return SANDY_ERR_UNSUPPORTED;
 }
 
@@ -196,7 +199,7 @@ SANDY_API int sandy_attention_prepare_pos(const void* proj, int ld, int q_off, i
     return sandy_attention_prepare_rot(proj, ld, q_off, k_off, v_off, n_tokens, n_heads, n_kv_heads, qk_dim, v_dim, pad_dim, q_gain,
                                        k_gain, eps, freq, rot_dims, positions, token_seq, block_table, max_blocks, k_cache, v_cache,
                                        page_stride, page_size, num_pages, write_cache, q_out, ld_q, gate_in, ld_gate, gate_out,
-                                       gate_scale, q_head_scale, v_unit_eps, per_head_norm, q_pos_coef, q_pos_every, 0, dtype, status,
+                                       gate_scale, q_head_scale, v_unit_eps, per_head_norm, q_pos_coef, q_pos_every, 0, 1.0f, dtype, status,
                                        stream);
 }
 

@@ -217,7 +217,7 @@ def _core_hash() -> str:
         with open(os.path.join(CORE_DIR, fname), "rb") as f:
             h.update(fname.encode())
             h.update(f.read())
-    for shared in ("sandy_kernels.h", "matrix_state.h"):
+    for shared in ("sandy_kernels.h", "matrix_state.h", "gated_linear.h", "attention_rules.h"):
         with open(os.path.join(CSRC_DIR, shared), "rb") as f:
             h.update(f.read())
     h.update(" ".join(CXX_FLAGS + LINK_FLAGS).encode())

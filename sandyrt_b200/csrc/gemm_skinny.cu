@@ -31,6 +31,9 @@
 // bfloat16, the same rounding point as the stand-alone norm kernel.  This trades a launch for
 // re-reading x (M x K floats, from L2) in every block, which pays while M is small.
 //
+// Several products of one shape in one launch (`ColumnGroups`): the weights stacked, the inputs side by side in a row of `a`;
+// columns [g * cols, (g + 1) * cols) of the output then read columns [g * K, (g + 1) * K) of the row.
+//
 // The warps' partial sums are added in a fixed order (warp 0, 1, ...), so a token's result
 // does not depend on what else is in the batch (rows of other tokens never enter its dot
 // products).
@@ -79,6 +82,11 @@ struct KVWrite {
     int* status;
 };
 
+// cols > 0 (a multiple of 16): every `cols` output columns read their input `a_step` elements further on in a row of `a`.
+struct ColumnGroups {
+    int cols, a_step;
+};
+
 struct NormArgs {
     const float* x;          // [M, K] float, row stride ldx
     const bf16* gamma;       // [K]
@@ -98,7 +106,7 @@ template <int MT, typename TC, bool FUSE_LN, int UNROLL, int RV>
 __global__ void __launch_bounds__(WARPS * 32, (UNROLL == 4 && RV <= 8 && MT == 1) ? 3 : ((MT > 1 && !FUSE_LN && UNROLL == 4) ? 2 : 1))
 gemm_skinny_kernel(const bf16* __restrict__ a, NormArgs norm, const bf16* __restrict__ w,
                    const bf16* __restrict__ bias, const float* residual, TC* out, int M, int N, int K, int lda,
-                   int ldw, int ldr, int ldc, int act, KVWrite kv) {
+                   int ldw, int ldr, int ldc, int act, KVWrite kv, ColumnGroups groups) {
     __shared__ float partial[WARPS][MT * 16][COLS + 1];
     extern __shared__ __align__(16) uint8_t xs_raw[];
     bf16* xs = reinterpret_cast<bf16*>(xs_raw);          // [MT*16][K + XPAD], fused norm only
@@ -107,6 +115,7 @@ gemm_skinny_kernel(const bf16* __restrict__ a, NormArgs norm, const bf16* __rest
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const int g = lane >> 2, t = lane & 3;
     const int n0 = blockIdx.x * COLS;
+    if (!FUSE_LN && groups.cols) a += (n0 / groups.cols) * groups.a_step;
     // this warp's contiguous slice of K, in whole chunks
     const int chunks = (K + KCHUNK - 1) / KCHUNK;
     const int per_warp = (chunks + WARPS - 1) / WARPS;
@@ -309,7 +318,7 @@ gemm_skinny_kernel(const bf16* __restrict__ a, NormArgs norm, const bf16* __rest
 template <int MT, bool FUSE_LN, int UNROLL, int RV>
 int launch2(const void* a, const NormArgs& norm, const void* w, const void* bias, const float* residual, void* out,
             int M, int N, int K, int lda, int ldw, int ldr, int ldc, int act, int out_dtype, const KVWrite& kv,
-            cudaStream_t stream) {
+            const ColumnGroups& groups, cudaStream_t stream) {
     const unsigned blocks = (unsigned)((N + COLS - 1) / COLS);
     const size_t smem = FUSE_LN ? ((size_t)MT * 16 * (K + XPAD) + 2 * (size_t)K) * sizeof(bf16) : 0;   // rows, gain, offset
     if (out_dtype == SANDY_F32) {
@@ -319,7 +328,7 @@ int launch2(const void* a, const NormArgs& norm, const void* w, const void* bias
             if (e != cudaSuccess) return (int)e;
         }
         return sandy_launch(kern, dim3(blocks), dim3(WARPS * 32), smem, stream, (const bf16*)a, norm, (const bf16*)w,
-                            (const bf16*)bias, residual, (float*)out, M, N, K, lda, ldw, ldr, ldc, act, kv);
+                            (const bf16*)bias, residual, (float*)out, M, N, K, lda, ldw, ldr, ldc, act, kv, groups);
     } else {
         auto kern = gemm_skinny_kernel<MT, bf16, FUSE_LN, UNROLL, RV>;
         if (smem > 40 * 1024) {
@@ -327,14 +336,14 @@ int launch2(const void* a, const NormArgs& norm, const void* w, const void* bias
             if (e != cudaSuccess) return (int)e;
         }
         return sandy_launch(kern, dim3(blocks), dim3(WARPS * 32), smem, stream, (const bf16*)a, norm, (const bf16*)w,
-                            (const bf16*)bias, residual, (bf16*)out, M, N, K, lda, ldw, ldr, ldc, act, kv);
+                            (const bf16*)bias, residual, (bf16*)out, M, N, K, lda, ldw, ldr, ldc, act, kv, groups);
     }
 }
 
 template <int MT, bool FUSE_LN, int RV>
 int launch1(const void* a, const NormArgs& norm, const void* w, const void* bias, const float* residual, void* out,
             int M, int N, int K, int lda, int ldw, int ldr, int ldc, int act, int out_dtype, const KVWrite& kv,
-            cudaStream_t stream) {
+            const ColumnGroups& groups, cudaStream_t stream) {
     // 16-byte pieces of one warp's K slice
     const int per_warp = ((K + KCHUNK - 1) / KCHUNK + WARPS - 1) / WARPS;
     // More blocks than SMs: what counts is how many blocks an SM holds, and the short rounds' 80 registers
@@ -343,21 +352,21 @@ int launch1(const void* a, const NormArgs& norm, const void* w, const void* bias
     // 1.89 / 2.23 ms).
     const bool crowded = MT == 1 && (N + COLS - 1) / COLS > sandy_sm_count();
     if (per_warp <= 4 || crowded)
-        return launch2<MT, FUSE_LN, 4, RV>(a, norm, w, bias, residual, out, M, N, K, lda, ldw, ldr, ldc, act, out_dtype, kv, stream);
+        return launch2<MT, FUSE_LN, 4, RV>(a, norm, w, bias, residual, out, M, N, K, lda, ldw, ldr, ldc, act, out_dtype, kv, groups, stream);
     if (per_warp <= 8 || MT > 1)
-        return launch2<MT, FUSE_LN, 8, RV>(a, norm, w, bias, residual, out, M, N, K, lda, ldw, ldr, ldc, act, out_dtype, kv, stream);
-    return launch2<MT, FUSE_LN, 16, RV>(a, norm, w, bias, residual, out, M, N, K, lda, ldw, ldr, ldc, act, out_dtype, kv, stream);
+        return launch2<MT, FUSE_LN, 8, RV>(a, norm, w, bias, residual, out, M, N, K, lda, ldw, ldr, ldc, act, out_dtype, kv, groups, stream);
+    return launch2<MT, FUSE_LN, 16, RV>(a, norm, w, bias, residual, out, M, N, K, lda, ldw, ldr, ldc, act, out_dtype, kv, groups, stream);
 }
 
 template <int MT, bool FUSE_LN>
 int launch(const void* a, const NormArgs& norm, const void* w, const void* bias, const float* residual, void* out,
            int M, int N, int K, int lda, int ldw, int ldr, int ldc, int act, int out_dtype, const KVWrite& kv,
-           cudaStream_t stream) {
+           const ColumnGroups& groups, cudaStream_t stream) {
     if (!FUSE_LN || K <= 512)
-        return launch1<MT, FUSE_LN, 4>(a, norm, w, bias, residual, out, M, N, K, lda, ldw, ldr, ldc, act, out_dtype, kv, stream);
+        return launch1<MT, FUSE_LN, 4>(a, norm, w, bias, residual, out, M, N, K, lda, ldw, ldr, ldc, act, out_dtype, kv, groups, stream);
     if (K <= 1024)
-        return launch1<MT, FUSE_LN, 8>(a, norm, w, bias, residual, out, M, N, K, lda, ldw, ldr, ldc, act, out_dtype, kv, stream);
-    return launch1<MT, FUSE_LN, 16>(a, norm, w, bias, residual, out, M, N, K, lda, ldw, ldr, ldc, act, out_dtype, kv, stream);
+        return launch1<MT, FUSE_LN, 8>(a, norm, w, bias, residual, out, M, N, K, lda, ldw, ldr, ldc, act, out_dtype, kv, groups, stream);
+    return launch1<MT, FUSE_LN, 16>(a, norm, w, bias, residual, out, M, N, K, lda, ldw, ldr, ldc, act, out_dtype, kv, groups, stream);
 }
 
 // ---- 17 to 64 rows and many columns: sixteen columns a block ------------------------------------
@@ -379,12 +388,13 @@ template <int MT, typename TC>
 __global__ void __launch_bounds__(WARPS * 32, 2)
 gemm_skinny_wide_kernel(const bf16* __restrict__ a, const bf16* __restrict__ w, const bf16* __restrict__ bias,
                         const float* residual, TC* out, int M, int N, int K, int lda, int ldw, int ldr, int ldc, int act,
-                        KVWrite kv) {
+                        KVWrite kv, ColumnGroups groups) {
     constexpr int UNROLL = 2;
     __shared__ float partial[WARPS][MT * 16][COLS2 + 1];
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const int g = lane >> 2, t = lane & 3;
     const int n0 = blockIdx.x * COLS2;
+    if (groups.cols) a += (n0 / groups.cols) * groups.a_step;
     const int chunks = (K + KCHUNK - 1) / KCHUNK;
     const int per_warp = (chunks + WARPS - 1) / WARPS;
     const int c_begin = warp * per_warp, c_end = min(chunks, c_begin + per_warp);
@@ -509,13 +519,13 @@ constexpr int WIDE_MIN_COLS = 1536;     // from here on half the blocks still fi
 
 template <int MT>
 int launch_wide(const void* a, const void* w, const void* bias, const float* residual, void* out, int M, int N, int K, int lda,
-                int ldw, int ldr, int ldc, int act, int out_dtype, const KVWrite& kv, cudaStream_t stream) {
+                int ldw, int ldr, int ldc, int act, int out_dtype, const KVWrite& kv, const ColumnGroups& groups, cudaStream_t stream) {
     const unsigned blocks = (unsigned)((N + COLS2 - 1) / COLS2);
     if (out_dtype == SANDY_F32)
         return sandy_launch(gemm_skinny_wide_kernel<MT, float>, dim3(blocks), dim3(WARPS * 32), 0, stream, (const bf16*)a,
-                            (const bf16*)w, (const bf16*)bias, residual, (float*)out, M, N, K, lda, ldw, ldr, ldc, act, kv);
+                            (const bf16*)w, (const bf16*)bias, residual, (float*)out, M, N, K, lda, ldw, ldr, ldc, act, kv, groups);
     return sandy_launch(gemm_skinny_wide_kernel<MT, bf16>, dim3(blocks), dim3(WARPS * 32), 0, stream, (const bf16*)a,
-                        (const bf16*)w, (const bf16*)bias, residual, (bf16*)out, M, N, K, lda, ldw, ldr, ldc, act, kv);
+                        (const bf16*)w, (const bf16*)bias, residual, (bf16*)out, M, N, K, lda, ldw, ldr, ldc, act, kv, groups);
 }
 
 // ---- a vocabulary projection: up to 16 rows, very many columns, nothing fused -------------------
@@ -629,20 +639,13 @@ SANDY_API int sandy_gemm_skinny_norm_limits(int* max_rows, int* max_k) {
     return SANDY_OK;
 }
 
-// Arguments as sandy_gemm_tc; M <= 64; K, lda, ldw multiples of 8; a and w 16-byte aligned.
-//
-// Fused norm: pass a = null and x (float [M, K], row stride ldx, 16-byte aligned, ldx % 4 == 0),
-// gamma, beta (bfloat16 [K], beta may be null), eps; M <= 16 and K <= 2048.
-// Key/value write: pass k_cache != null with the cache description of attention.cu; columns
-// [q_cols, q_cols + kv_cols) of the product are keys, the next kv_cols are values, and row m
-// belongs to position positions[m] of request token_seq[m].  out must be bfloat16 then.
-SANDY_API int sandy_gemm_skinny(const void* a, const float* x, int ldx, const void* gamma, const void* beta,
+static int gemm_skinny_any(const void* a, const float* x, int ldx, const void* gamma, const void* beta,
                                 float eps, const void* w, const void* bias, const float* residual, void* out,
                                 int M, int N, int K, int lda, int ldw, int ldr, int ldc, int act, int out_dtype,
                                 void* k_cache, void* v_cache, long long page_stride, const int* block_table,
                                 int max_blocks, const int* token_seq, const int* positions, int q_cols,
                                 int kv_cols, int head_dim, int page_size, int num_pages, int* status,
-                                cudaStream_t stream) {
+                                const ColumnGroups& groups, cudaStream_t stream) {
     if (M == 0 || N == 0) return SANDY_OK;
     const bool fuse = a == nullptr;
     if ((!a && !x) || !w || !out || K <= 0) return SANDY_ERR_ARGUMENT;
@@ -664,18 +667,48 @@ SANDY_API int sandy_gemm_skinny(const void* a, const float* x, int ldx, const vo
             kv_cols % head_dim != 0 || q_cols + 2 * kv_cols != N || page_size <= 0)
             return SANDY_ERR_ARGUMENT;
     }
-    if (!fuse && !k_cache && !bias && !residual && act == SANDY_ACT_NONE && M <= 16 && K <= WALK_MAX_K &&
+    if (!fuse && !k_cache && !groups.cols && !bias && !residual && act == SANDY_ACT_NONE && M <= 16 && K <= WALK_MAX_K &&
         (N + COLS - 1) / COLS >= WALK_MIN_GROUPS) {
         if (out_dtype == SANDY_F32) return launch_walk<float>(a, w, out, M, N, K, lda, ldw, ldc, stream);
         return launch_walk<bf16>(a, w, out, M, N, K, lda, ldw, ldc, stream);
     }
-    if (fuse) return launch<1, true>(a, norm, w, bias, residual, out, M, N, K, lda, ldw, ldr, ldc, act, out_dtype, kv, stream);
-    if (M <= 16) return launch<1, false>(a, norm, w, bias, residual, out, M, N, K, lda, ldw, ldr, ldc, act, out_dtype, kv, stream);
+    if (fuse) return launch<1, true>(a, norm, w, bias, residual, out, M, N, K, lda, ldw, ldr, ldc, act, out_dtype, kv, groups, stream);
+    if (M <= 16) return launch<1, false>(a, norm, w, bias, residual, out, M, N, K, lda, ldw, ldr, ldc, act, out_dtype, kv, groups, stream);
     if (N >= WIDE_MIN_COLS) {
-        if (M <= 32) return launch_wide<2>(a, w, bias, residual, out, M, N, K, lda, ldw, ldr, ldc, act, out_dtype, kv, stream);
-        if (M <= 48) return launch_wide<3>(a, w, bias, residual, out, M, N, K, lda, ldw, ldr, ldc, act, out_dtype, kv, stream);
-        return launch_wide<4>(a, w, bias, residual, out, M, N, K, lda, ldw, ldr, ldc, act, out_dtype, kv, stream);
+        if (M <= 32) return launch_wide<2>(a, w, bias, residual, out, M, N, K, lda, ldw, ldr, ldc, act, out_dtype, kv, groups, stream);
+        if (M <= 48) return launch_wide<3>(a, w, bias, residual, out, M, N, K, lda, ldw, ldr, ldc, act, out_dtype, kv, groups, stream);
+        return launch_wide<4>(a, w, bias, residual, out, M, N, K, lda, ldw, ldr, ldc, act, out_dtype, kv, groups, stream);
     }
-    if (M <= 32) return launch<2, false>(a, norm, w, bias, residual, out, M, N, K, lda, ldw, ldr, ldc, act, out_dtype, kv, stream);
-    return launch<4, false>(a, norm, w, bias, residual, out, M, N, K, lda, ldw, ldr, ldc, act, out_dtype, kv, stream);
+    if (M <= 32) return launch<2, false>(a, norm, w, bias, residual, out, M, N, K, lda, ldw, ldr, ldc, act, out_dtype, kv, groups, stream);
+    return launch<4, false>(a, norm, w, bias, residual, out, M, N, K, lda, ldw, ldr, ldc, act, out_dtype, kv, groups, stream);
+}
+
+// Arguments as sandy_gemm_tc; M <= 64; K, lda, ldw multiples of 8; a and w 16-byte aligned.
+//
+// Fused norm: pass a = null and x (float [M, K], row stride ldx, 16-byte aligned, ldx % 4 == 0),
+// gamma, beta (bfloat16 [K], beta may be null), eps; M <= 16 and K <= 2048.
+// Key/value write: pass k_cache != null with the cache description of attention.cu; columns
+// [q_cols, q_cols + kv_cols) of the product are keys, the next kv_cols are values, and row m
+// belongs to position positions[m] of request token_seq[m].  out must be bfloat16 then.
+SANDY_API int sandy_gemm_skinny(const void* a, const float* x, int ldx, const void* gamma, const void* beta,
+                                float eps, const void* w, const void* bias, const float* residual, void* out,
+                                int M, int N, int K, int lda, int ldw, int ldr, int ldc, int act, int out_dtype,
+                                void* k_cache, void* v_cache, long long page_stride, const int* block_table,
+                                int max_blocks, const int* token_seq, const int* positions, int q_cols,
+                                int kv_cols, int head_dim, int page_size, int num_pages, int* status,
+                                cudaStream_t stream) {
+    return gemm_skinny_any(a, x, ldx, gamma, beta, eps, w, bias, residual, out, M, N, K, lda, ldw, ldr, ldc, act, out_dtype, k_cache,
+                           v_cache, page_stride, block_table, max_blocks, token_seq, positions, q_cols, kv_cols, head_dim, page_size,
+                           num_pages, status, ColumnGroups{0, 0}, stream);
+}
+
+// n_groups products of one shape in one launch: out[m, g * cols + n] = sum_k a[m, g * K + k] w[g * cols + n, k]; cols a multiple
+// of 16; a: bfloat16 [M, n_groups * K].
+SANDY_API int sandy_gemm_skinny_groups(const void* a, const void* w, void* out, int M, int n_groups, int cols, int K, int lda,
+                                       int ldw, int ldc, int out_dtype, cudaStream_t stream) {
+    if (!a) return SANDY_ERR_ARGUMENT;
+    if (n_groups <= 0 || cols <= 0 || cols % 16 || lda < n_groups * K) return SANDY_ERR_UNSUPPORTED;
+    return gemm_skinny_any(a, nullptr, 0, nullptr, nullptr, 0.0f, w, nullptr, nullptr, out, M, n_groups * cols, K, lda, ldw, 0, ldc,
+                           SANDY_ACT_NONE, out_dtype, nullptr, nullptr, 0, nullptr, 0, nullptr, nullptr, 0, 0, 0, 0, 0, nullptr,
+                           ColumnGroups{cols, K}, stream);
 }

@@ -43,22 +43,23 @@ __device__ __forceinline__ float silu_f(float z) { return z / (1.0f + expf(-z));
 // ---- gated delta rule: what comes before the recurrence ---------------------------------------------------
 // Per token: the short causal convolution of the q, k and v channels (taps from the step's earlier tokens
 // or, before the step's start, from the tail kept in the state), silu, unit vectors per q/k head (q also
-// times q_scale), and the two gates.  One block per token.
+// times q_scale), and the two gates (none with null `gates`).  One block per token.  With `keep` (every request brings one
+// token) the tail moves on by the token in the same launch.
 template <typename T>
 __global__ void __launch_bounds__(256)
 delta_prepare_kernel(const T* __restrict__ proj, int ld, const float* __restrict__ taps, int n_taps,
                      const float* __restrict__ gates, int ld_gates, const float* __restrict__ a_log,
-                     const float* __restrict__ dt_bias, const float* __restrict__ state, long long state_stride,
+                     const float* __restrict__ dt_bias, float* __restrict__ state, long long state_stride,
                      long long tail_off, const int* __restrict__ token_seq, const int* __restrict__ q_start,
                      const int* __restrict__ seq_slots, float* __restrict__ qkv, int ld_qkv, float* __restrict__ bg,
-                     int n_heads, int n_qk_heads, int qk_dim, int v_dim, float q_scale) {
+                     int n_heads, int n_qk_heads, int qk_dim, int v_dim, float q_scale, int keep) {
     extern __shared__ float act[];                    // [channels]
     const int t = blockIdx.x;
     const int qk = n_qk_heads * qk_dim;
     const int channels = 2 * qk + n_heads * v_dim;
     const int s = token_seq[t];
     const int i_in_step = t - q_start[s];
-    const float* tail = state + (long long)seq_slots[s] * state_stride + tail_off;      // [n_taps - 1][channels]
+    float* tail = state + (long long)seq_slots[s] * state_stride + tail_off;      // [n_taps - 1][channels]
     pdl_wait();
     pdl_launch_dependents();
     for (int c = threadIdx.x; c < channels; c += blockDim.x) {
@@ -70,6 +71,10 @@ delta_prepare_kernel(const T* __restrict__ proj, int ld, const float* __restrict
             y = fmaf(taps[(size_t)c * n_taps + j], x, y);
         }
         act[c] = silu_f(y);
+        if (keep && n_taps > 1) {                     // this thread alone reads and writes its channel of the tail
+            for (int j = 0; j + 2 < n_taps; j++) tail[(size_t)j * channels + c] = tail[(size_t)(j + 1) * channels + c];
+            tail[(size_t)(n_taps - 2) * channels + c] = to_f32(proj[(size_t)t * ld + c]);
+        }
     }
     __syncthreads();
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, n_warps = blockDim.x >> 5;
@@ -83,6 +88,7 @@ delta_prepare_kernel(const T* __restrict__ proj, int ld, const float* __restrict
         for (int i = lane; i < qk_dim; i += 32) out[head * qk_dim + i] = x[i] * inv;
     }
     for (int c = 2 * qk + threadIdx.x; c < channels; c += blockDim.x) out[c] = act[c];
+    if (!gates) return;
     for (int h = threadIdx.x; h < n_heads; h += blockDim.x) {
         const float b = gates[(size_t)t * ld_gates + h], a = gates[(size_t)t * ld_gates + n_heads + h];
         bg[(size_t)t * 2 * n_heads + h] = 1.0f / (1.0f + expf(-b));
@@ -850,13 +856,15 @@ SANDY_API long long sandy_mlstm_state_floats(int n_heads, int qk_dim, int v_dim)
     return (long long)n_heads * v_dim * qk_dim + (long long)n_heads * Z * qk_dim + (long long)n_heads * Z;
 }
 
-SANDY_API int sandy_delta_prepare(const void* proj, int ld, int dtype, const float* taps, int n_taps, const float* gates,
-                                  int ld_gates, const float* a_log, const float* dt_bias, const float* state,
+// gates null: no gates are formed (a_log, dt_bias and bg are then not read or written).  keep != 0, only in steps in which every
+// request brings one token: the convolution's tail moves on by it (sandy_conv_tail otherwise).
+SANDY_API int sandy_delta_prepare_keep(const void* proj, int ld, int dtype, const float* taps, int n_taps, const float* gates,
+                                  int ld_gates, const float* a_log, const float* dt_bias, float* state,
                                   long long state_stride, long long tail_off, const int* token_seq, const int* q_start,
                                   const int* seq_slots, float* qkv, int ld_qkv, float* bg, int n_tokens, int n_heads,
-                                  int n_qk_heads, int qk_dim, int v_dim, float q_scale, cudaStream_t stream) {
+                                  int n_qk_heads, int qk_dim, int v_dim, float q_scale, int keep, cudaStream_t stream) {
     if (n_tokens == 0) return SANDY_OK;
-    if (!proj || !taps || !gates || !a_log || !dt_bias || !state || !qkv || !bg) return SANDY_ERR_ARGUMENT;
+    if (!proj || !taps || (gates && (!a_log || !dt_bias || !bg)) || !state || !qkv) return SANDY_ERR_ARGUMENT;
     if (n_taps < 1 || n_taps > MAX_TAPS || n_qk_heads <= 0 || n_heads % n_qk_heads) return SANDY_ERR_UNSUPPORTED;
     const size_t smem = (size_t)(2 * n_qk_heads * qk_dim + n_heads * v_dim) * sizeof(float);
     if (smem > 200 * 1024) return SANDY_ERR_UNSUPPORTED;
@@ -868,12 +876,23 @@ SANDY_API int sandy_delta_prepare(const void* proj, int ld, int dtype, const flo
         }                                                                                                               \
         return sandy_launch(delta_prepare_kernel<TT>, dim3(n_tokens), dim3(256), smem, stream, (const TT*)proj, ld, taps, \
                             n_taps, gates, ld_gates, a_log, dt_bias, state, state_stride, tail_off, token_seq, q_start,  \
-                            seq_slots, qkv, ld_qkv, bg, n_heads, n_qk_heads, qk_dim, v_dim, q_scale);                   \
+                            seq_slots, qkv, ld_qkv, bg, n_heads, n_qk_heads, qk_dim, v_dim, q_scale, keep);             \
     } while (0)
     if (dtype == SANDY_F32) GO(float);
     if (dtype == SANDY_BF16) GO(bf16);
 #undef GO
     return SANDY_ERR_UNSUPPORTED;
+}
+
+SANDY_API int sandy_delta_prepare(const void* proj, int ld, int dtype, const float* taps, int n_taps, const float* gates,
+                                  int ld_gates, const float* a_log, const float* dt_bias, const float* state,
+                                  long long state_stride, long long tail_off, const int* token_seq, const int* q_start,
+                                  const int* seq_slots, float* qkv, int ld_qkv, float* bg, int n_tokens, int n_heads,
+                                  int n_qk_heads, int qk_dim, int v_dim, float q_scale, cudaStream_t stream) {
+    if (n_tokens && !gates) return SANDY_ERR_ARGUMENT;
+    return sandy_delta_prepare_keep(proj, ld, dtype, taps, n_taps, gates, ld_gates, a_log, dt_bias, const_cast<float*>(state), state_stride,
+                                    tail_off, token_seq, q_start, seq_slots, qkv, ld_qkv, bg, n_tokens, n_heads, n_qk_heads, qk_dim,
+                                    v_dim, q_scale, 0, stream);
 }
 
 SANDY_API int sandy_conv_tail(const void* proj, int ld, int dtype, int channels, int n_taps, float* state,

@@ -477,7 +477,7 @@ def softcap(x, cap: float) -> None:
 def rmsnorm_shift(x, gain, mix, state, token_seq, q_start, seq_slots, out, *, eps: float) -> None:
     """Token shift behind an RMS norm: h[t] = x[t] / rms(x[t]) * gain; out[t] = h[t] + (h[t-1] - h[t]) * mix, where the h
     before a request's first token of the step is its row of `state` (float32 [slots, >= width]); afterwards every
-    request's row holds the h of its last token."""
+    request's row holds the h of its last token.  mix [width], or [n, width] for n results side by side in out [T, n * width]."""
     _cuda(x, gain, mix, state, token_seq, q_start, seq_slots, out)
     for t, n in ((x, "x"), (gain, "gain"), (mix, "mix")):
         _f32(t, n)
@@ -487,8 +487,8 @@ def rmsnorm_shift(x, gain, mix, state, token_seq, q_start, seq_slots, out, *, ep
     T, W = x.shape
     S = seq_slots.numel()
     lib = load_library("rmsnorm")
-    _check(lib.sandy_rmsnorm_shift(_p(x), ctypes.c_int(x.stride(0)), _p(gain), _p(mix), _p(state), ctypes.c_longlong(state.stride(0)),
-                                   _p(token_seq), _p(q_start), _p(seq_slots), _p(out), ctypes.c_int(out.stride(0)), ctypes.c_int(T),
+    _check(lib.sandy_rmsnorm_shifts(_p(x), ctypes.c_int(x.stride(0)), _p(gain), _p(mix), ctypes.c_int(mix.numel() // W), _p(state),
+                                   ctypes.c_longlong(state.stride(0)), _p(token_seq), _p(q_start), _p(seq_slots), _p(out), ctypes.c_int(out.stride(0)), ctypes.c_int(T),
                                    ctypes.c_int(W), ctypes.c_float(eps), ctypes.c_int(_dt(out)), _stream()), "rmsnorm_shift")
     _check(lib.sandy_rmsnorm_keep(_p(x), ctypes.c_int(x.stride(0)), _p(gain), _p(state), ctypes.c_longlong(state.stride(0)), _p(q_start),
                                   _p(seq_slots), ctypes.c_int(S), ctypes.c_int(W), ctypes.c_float(eps), _stream()), "rmsnorm_keep")
@@ -744,19 +744,22 @@ def gated_group_norm(y, z, gain, out, *, groups: int, eps: float) -> None:
 
 
 def attention_prepare(proj, k_cache, v_cache, block_table, token_seq, positions, q_out, *, n_heads: int, qk_dim: int, v_dim: int,
-                      freq=None, interleaved: bool = False, write_cache: bool = True) -> None:
-    """Queries, keys and values out of a projection [T, H * qk_dim | Hkv * qk_dim | Hkv * v_dim | ...]: the first
-    2 * len(freq) entries of every query and key head turn (halves, or neighbours with `interleaved`), keys and values go
-    into their pages, queries into q_out [T, H * D], heads padded with zeros to the cache's head size D."""
+                      freq=None, interleaved: bool = False, write_cache: bool = True, rot_scale: float = 1.0,
+                      values_are_keys: bool = False, head_scale=None) -> None:
+    """Queries, keys and values out of a projection [T, H * qk_dim | Hkv * qk_dim | Hkv * v_dim | ...] (without values where they
+    are the keys before the rotation): the first 2 * len(freq) entries of every query and key head turn (halves, or neighbours
+    with `interleaved`; cosine and sine times rot_scale), keys and values go into their pages, queries into q_out [T, H * D],
+    heads padded with zeros to the cache's head size D.  head_scale: (float32 [T, H], factor) that is filled with the factor."""
     _cuda(proj, k_cache, v_cache, block_table, token_seq, positions, q_out, freq)
     hkv, ps, d, page_stride, num_pages = _cache_args(k_cache, v_cache)
     null, i = ctypes.c_void_p(0), ctypes.c_int
     code = load_library("attention_prepare").sandy_attention_prepare_rot(
-        _p(proj), i(proj.stride(0)), i(0), i(n_heads * qk_dim), i((n_heads + hkv) * qk_dim), i(proj.shape[0]), i(n_heads), i(hkv), i(qk_dim),
+        _p(proj), i(proj.stride(0)), i(0), i(n_heads * qk_dim), i((n_heads + (0 if values_are_keys else hkv)) * qk_dim), i(proj.shape[0]), i(n_heads), i(hkv), i(qk_dim),
         i(v_dim), i(d), null, null, ctypes.c_float(0.0), _p(freq), i(0 if freq is None else 2 * freq.numel()), _p(positions), _p(token_seq),
         _p(block_table), i(block_table.shape[1]), _p(k_cache), _p(v_cache), ctypes.c_longlong(page_stride), i(ps), i(num_pages),
-        i(1 if write_cache else 0), _p(q_out), i(q_out.stride(0)), null, i(0), null, ctypes.c_float(1.0), null, ctypes.c_float(0.0), i(0),
-        ctypes.c_float(0.0), i(0), i(1 if interleaved else 0), i(_dt(proj)), _p(kernel_status(proj.device)), _stream())
+        i(1 if write_cache else 0), _p(q_out), i(q_out.stride(0)), null, i(0), _p(head_scale[0] if head_scale else None),
+        ctypes.c_float(head_scale[1] if head_scale else 1.0), null, ctypes.c_float(0.0), i(0),
+        ctypes.c_float(0.0), i(0), i(1 if interleaved else 0), ctypes.c_float(rot_scale), i(_dt(proj)), _p(kernel_status(proj.device)), _stream())
     _check(code, "attention_prepare")
 
 
@@ -778,6 +781,52 @@ def gla_scan(proj, low, w2t, bias, state, q_start, seq_slots, out, *, n_heads: i
         scratch = torch.full((int(floats),), float("nan"), dtype=torch.float32, device=proj.device)
         _check(lib.sandy_gla_chunk_scan(*head, _p(scratch), i(T), i(S), i(max_q_len), i(n_heads), i(qk_dim), i(v_dim), i(chunked_from),
                                         _stream()), "gla_chunk_scan")
+
+
+class _FadeRule(ctypes.Structure):
+    """SandyFadeRule of gated_linear.h."""
+    _fields_ = [("kind", ctypes.c_int), ("decay", ctypes.c_int), ("inv_tau", ctypes.c_float), ("tanh_low", ctypes.c_int),
+                ("a_log", ctypes.c_void_p), ("bonus", ctypes.c_void_p), ("beta", ctypes.c_void_p), ("ld_beta", ctypes.c_int),
+                ("n_qk_heads", ctypes.c_int)]
+
+
+FADE_KINDS = {"add": 0, "bonus": 1, "delta": 2}
+DECAY_FORMS = {"logsigmoid": 0, "exp": 1, "softplus": 2}
+
+
+def fade_scan(proj, low, w2t, bias, state, q_start, seq_slots, out, *, n_heads: int, qk_dim: int, v_dim: int, q_scale: float,
+              kind: str = "add", decay: str = "logsigmoid", tau: float = 1.0, tanh_low: bool = False, a_log=None, bonus=None, beta=None,
+              n_qk_heads: int = 0, chunked_from: int = 0, max_q_len: int = 0) -> None:
+    """A recurrence with a decay per key channel (gated_linear.cu).  proj [T, Hq * qk_dim | Hq * qk_dim | H * v_dim | ...] (q, k, v);
+    low float32 [T, rank]; w2t float32 [rank, H * qk_dim]; bias float32 [H * qk_dim]; `state` float32 [slots, >= H * v_dim *
+    qk_dim]; a_log [H] (decay "softplus"), bonus [H * qk_dim] (kind "bonus"), beta [T, H] (kind "delta"), all float32.
+    Requests with chunked_from tokens or more take the chunked kernels (0: none)."""
+    _cuda(proj, low, w2t, bias, state, q_start, seq_slots, out, a_log, bonus, beta)
+    lib, i, f = load_library("gated_linear"), ctypes.c_int, ctypes.c_float
+    S, T, hq = seq_slots.numel(), proj.shape[0], n_qk_heads or n_heads
+    rule = _FadeRule(FADE_KINDS[kind], DECAY_FORMS[decay], 1.0 / tau, int(tanh_low), _p(a_log), _p(bonus), _p(beta),
+                     0 if beta is None else beta.stride(0), n_qk_heads)
+    head = (_p(proj), i(proj.stride(0)), i(_dt(proj)), i(0), i(hq * qk_dim), i(2 * hq * qk_dim), _p(low), i(low.stride(0)),
+            i(low.shape[1]), _p(w2t), _p(bias), ctypes.byref(rule), f(q_scale), _p(state), ctypes.c_longlong(state.stride(0)),
+            _p(q_start), _p(seq_slots), _p(out), i(out.stride(0)))
+    _check(lib.sandy_fade_scan(*head, i(S), i(n_heads), i(qk_dim), i(v_dim), i(chunked_from), _stream()), "fade_scan")
+    if chunked_from:
+        lib.sandy_fade_scratch_floats.restype = ctypes.c_longlong
+        floats = lib.sandy_fade_scratch_floats(i(FADE_KINDS[kind]), i(T), i(S), i(n_heads), i(qk_dim), i(v_dim))
+        scratch = torch.full((int(floats),), float("nan"), dtype=torch.float32, device=proj.device)
+        _check(lib.sandy_fade_chunk_scan(*head, _p(scratch), i(T), i(S), i(max_q_len), i(n_heads), i(qk_dim), i(v_dim), i(chunked_from),
+                                         _stream()), "fade_chunk_scan")
+
+
+def gemm_skinny_groups(a, w, out, *, n_groups: int) -> None:
+    """Products of one shape in one launch, up to 64 rows: columns g of n_groups equal column ranges of out = the g-th range of a
+    times the g-th range of w's rows.  a bfloat16 [M, n_groups * K], w bfloat16 [n_groups * N, K]."""
+    _cuda(a, w, out)
+    i = ctypes.c_int
+    code = load_library("gemm_skinny").sandy_gemm_skinny_groups(
+        _p(a), _p(w), _p(out), i(a.shape[0]), i(n_groups), i(w.shape[0] // n_groups), i(w.shape[1]), i(a.stride(0)), i(w.stride(0)),
+        i(out.stride(0)), i(_dt(out)), _stream())
+    _check(code, "gemm_skinny_groups")
 
 
 def sample(logits, out_tokens, *, temperature=None, top_k=None, top_p=None, uniform=None, status=None,

@@ -14,7 +14,9 @@
 //                                                                                    token before; the h before a
 //                                                                                    request's first token of the
 //                                                                                    step is its state row, zeros at
-//                                                                                    its very first token)
+//                                                                                    its very first token); with
+//                                                                                    several rows of mix, the results
+//                                                                                    side by side in one row of out
 //   sandy_rmsnorm_keep   state[slot of s] = norm(x[last token of s]) * gain          for requests with several tokens
 //
 // The mean is over the row (or the head) with eps inside the root.  The input is float32 (the residual
@@ -121,7 +123,7 @@ __global__ void __launch_bounds__(256)
 rmsnorm_shift_kernel(const float* __restrict__ x, int ldx, const float* __restrict__ gain, const float* __restrict__ mix,
                      float* __restrict__ state, long long state_stride, const int* __restrict__ token_seq,
                      const int* __restrict__ q_start, const int* __restrict__ seq_slots, TO* __restrict__ out, int ldo,
-                     int width, float eps) {
+                     int width, int n_mix, float eps) {
     __shared__ float scratch[32], scratch_prev[32];
     const int t = blockIdx.x;
     const int s = token_seq[t];                      // the step's index arrays were staged before the step
@@ -143,7 +145,7 @@ rmsnorm_shift_kernel(const float* __restrict__ x, int ldx, const float* __restri
         const float g = gain ? gain[e] : 1.0f;
         const float h = row[e] * inv * g;
         const float before = t > first ? prow[e] * inv_prev * g : srow[e];
-        orow[e] = from_f32<TO>(h + (before - h) * mix[e]);
+        for (int j = 0; j < n_mix; j++) orow[(size_t)j * width + e] = from_f32<TO>(h + (before - h) * mix[(size_t)j * width + e]);
         if (first == last) srow[e] = h;
     }
 }
@@ -156,7 +158,7 @@ __global__ void __launch_bounds__(256)
 rmsnorm_shift_reg_kernel(const float* __restrict__ x, int ldx, const float* __restrict__ gain, const float* __restrict__ mix,
                          float* __restrict__ state, long long state_stride, const int* __restrict__ token_seq,
                          const int* __restrict__ q_start, const int* __restrict__ seq_slots, TO* __restrict__ out, int ldo,
-                         int width, float eps) {
+                         int width, int n_mix, float eps) {
     __shared__ float scratch[32], scratch_prev[32];
     const int t = blockIdx.x;
     const int s = token_seq[t];
@@ -197,6 +199,7 @@ rmsnorm_shift_reg_kernel(const float* __restrict__ x, int ldx, const float* __re
             const float h = v[i] * inv * g[i];
             const float before = inside ? p[i] * inv_prev * g[i] : p[i];
             orow[e] = from_f32<TO>(h + (before - h) * m[i]);
+            for (int j = 1; j < n_mix; j++) orow[(size_t)j * width + e] = from_f32<TO>(h + (before - h) * mix[(size_t)j * width + e]);
             if (first == last) srow[e] = h;
         }
     }
@@ -205,16 +208,16 @@ rmsnorm_shift_reg_kernel(const float* __restrict__ x, int ldx, const float* __re
 template <typename TO>
 int launch_shift(const float* x, int ldx, const float* gain, const float* mix, float* state, long long state_stride,
                  const int* token_seq, const int* q_start, const int* seq_slots, TO* out, int ldo, int n_tokens, int width,
-                 float eps, cudaStream_t stream) {
+                 int n_mix, float eps, cudaStream_t stream) {
     const int threads = width >= 1024 ? 256 : 128;
 #define CASE(NV)                                                                                                          \
     if (width <= threads * NV)                                                                                            \
         return sandy_launch(rmsnorm_shift_reg_kernel<TO, NV>, dim3(n_tokens), dim3(threads), 0, stream, x, ldx, gain, mix, \
-                            state, state_stride, token_seq, q_start, seq_slots, out, ldo, width, eps)
+                            state, state_stride, token_seq, q_start, seq_slots, out, ldo, width, n_mix, eps)
     CASE(2); CASE(4); CASE(6); CASE(8); CASE(16);
 #undef CASE
     return sandy_launch(rmsnorm_shift_kernel<TO>, dim3(n_tokens), dim3(threads), 0, stream, x, ldx, gain, mix, state,
-                        state_stride, token_seq, q_start, seq_slots, out, ldo, width, eps);
+                        state_stride, token_seq, q_start, seq_slots, out, ldo, width, n_mix, eps);
 }
 
 // A block per request of the step; requests with one token were served by the kernel above.
@@ -331,22 +334,30 @@ SANDY_API int sandy_head_norm_gate(const float* o, int ldo, const float* gain, i
     return SANDY_ERR_UNSUPPORTED;
 }
 
-// x: float32 [n_tokens, width] (pitch ldx); gain: float32 [width] or null; mix: float32 [width]; state: float32 rows of
+// x: float32 [n_tokens, width] (pitch ldx); gain: float32 [width] or null; mix: float32 [n_mix, width]; state: float32 rows of
 // `state_stride` floats, one per state slot, the first `width` of which hold the request's last h; out: [n_tokens,
-// width] of out_dtype.  token_seq [n_tokens], q_start [n_seqs + 1], seq_slots [n_seqs]: the step's index arrays.
-SANDY_API int sandy_rmsnorm_shift(const float* x, int ldx, const float* gain, const float* mix, float* state,
-                                  long long state_stride, const int* token_seq, const int* q_start, const int* seq_slots,
-                                  void* out, int ldo, int n_tokens, int width, float eps, int out_dtype, cudaStream_t stream) {
+// n_mix * width] of out_dtype.  token_seq [n_tokens], q_start [n_seqs + 1], seq_slots [n_seqs]: the step's index arrays.
+SANDY_API int sandy_rmsnorm_shifts(const float* x, int ldx, const float* gain, const float* mix, int n_mix, float* state,
+                                   long long state_stride, const int* token_seq, const int* q_start, const int* seq_slots,
+                                   void* out, int ldo, int n_tokens, int width, float eps, int out_dtype, cudaStream_t stream) {
     if (n_tokens == 0) return SANDY_OK;
-    if (!x || !mix || !state || !token_seq || !q_start || !seq_slots || !out || width <= 0 || state_stride < width)
+    if (!x || !mix || !state || !token_seq || !q_start || !seq_slots || !out || width <= 0 || n_mix <= 0 || state_stride < width)
         return SANDY_ERR_ARGUMENT;
     if (out_dtype == SANDY_F32)
         return launch_shift(x, ldx, gain, mix, state, state_stride, token_seq, q_start, seq_slots, (float*)out, ldo, n_tokens,
-                            width, eps, stream);
+                            width, n_mix, eps, stream);
     if (out_dtype == SANDY_BF16)
         return launch_shift(x, ldx, gain, mix, state, state_stride, token_seq, q_start, seq_slots, (bf16*)out, ldo, n_tokens,
-                            width, eps, stream);
+                            width, n_mix, eps, stream);
     return SANDY_ERR_UNSUPPORTED;
+}
+
+// One mix.
+SANDY_API int sandy_rmsnorm_shift(const float* x, int ldx, const float* gain, const float* mix, float* state,
+                                  long long state_stride, const int* token_seq, const int* q_start, const int* seq_slots,
+                                  void* out, int ldo, int n_tokens, int width, float eps, int out_dtype, cudaStream_t stream) {
+    return sandy_rmsnorm_shifts(x, ldx, gain, mix, 1, state, state_stride, token_seq, q_start, seq_slots, out, ldo, n_tokens, width, eps,
+                                out_dtype, stream);
 }
 
 // Runs behind sandy_rmsnorm_shift in steps that hold a request with more than one token.

@@ -10,6 +10,7 @@
 #include <cuda_runtime.h>
 
 #include "attention_rules.h"
+#include "gated_linear.h"
 #include "matrix_state.h"
 
 #ifdef __cplusplus
@@ -50,6 +51,9 @@ int sandy_gemm_skinny(const void* a, const float* x, int ldx, const void* gamma,
                       int ldc, int act, int out_dtype, void* k_cache, void* v_cache, long long page_stride,
                       const int* block_table, int max_blocks, const int* token_seq, const int* positions, int q_cols,
                       int kv_cols, int head_dim, int page_size, int num_pages, int* status, cudaStream_t stream);
+
+int sandy_gemm_skinny_groups(const void* a, const void* w, void* out, int M, int n_groups, int cols, int K, int lda, int ldw,
+                             int ldc, int out_dtype, cudaStream_t stream);
 
 /* gemm_small.cu */
 int sandy_gemm_small_splits(int N, int K);
@@ -252,10 +256,20 @@ int sandy_attention_prepare_rot(const void* proj, int ld, int q_off, int k_off, 
                                 const int* block_table, int max_blocks, void* k_cache, void* v_cache, long long page_stride,
                                 int page_size, int num_pages, int write_cache, void* q_out, int ld_q, const float* gate_in,
                                 int ld_gate, float* gate_out, float gate_scale, const float* q_head_scale, float v_unit_eps,
-                                int per_head_norm, float q_pos_coef, int q_pos_every, int interleaved, int dtype, int* status,
+                                int per_head_norm, float q_pos_coef, int q_pos_every, int interleaved, float rot_scale, int dtype, int* status,
                                 cudaStream_t stream);
 
 /* gated_linear.cu */
+int sandy_fade_scan(const void* proj, int ld, int dtype, int q_off, int k_off, int v_off, const float* low, int ld_low, int rank,
+                    const float* w2t, const float* bias, const SandyFadeRule* rule, float q_scale, float* state,
+                    long long state_stride, const int* q_start, const int* seq_slots, float* out, int ld_out, int n_seqs, int n_heads,
+                    int qk_dim, int v_dim, int long_from, cudaStream_t stream);
+long long sandy_fade_scratch_floats(int kind, int n_tokens, int n_seqs, int n_heads, int qk_dim, int v_dim);
+int sandy_fade_chunk_scan(const void* proj, int ld, int dtype, int q_off, int k_off, int v_off, const float* low, int ld_low, int rank,
+                          const float* w2t, const float* bias, const SandyFadeRule* rule, float q_scale, float* state,
+                          long long state_stride, const int* q_start, const int* seq_slots, float* out, int ld_out, float* scratch,
+                          int n_tokens, int n_seqs, int max_q_len, int n_heads, int qk_dim, int v_dim, int long_from,
+                          cudaStream_t stream);
 int sandy_gla_scan(const void* proj, int ld, int dtype, int q_off, int k_off, int v_off, const float* low, int ld_low, int rank,
                    const float* w2t, const float* bias, float inv_tau, float q_scale, float* state, long long state_stride,
                    const int* q_start, const int* seq_slots, float* out, int ld_out, int n_seqs, int n_heads, int qk_dim, int v_dim,
@@ -267,6 +281,9 @@ int sandy_gla_chunk_scan(const void* proj, int ld, int dtype, int q_off, int k_o
                          int max_q_len, int n_heads, int qk_dim, int v_dim, int long_from, cudaStream_t stream);
 
 /* rmsnorm.cu */
+int sandy_rmsnorm_shifts(const float* x, int ldx, const float* gain, const float* mix, int n_mix, float* state, long long state_stride,
+                         const int* token_seq, const int* q_start, const int* seq_slots, void* out, int ldo, int n_tokens, int width,
+                         float eps, int out_dtype, cudaStream_t stream);
 int sandy_rmsnorm_shift(const float* x, int ldx, const float* gain, const float* mix, float* state, long long state_stride,
                         const int* token_seq, const int* q_start, const int* seq_slots, void* out, int ldo, int n_tokens,
                         int width, float eps, int out_dtype, cudaStream_t stream);
@@ -366,6 +383,11 @@ int sandy_gated_group_norm(const float* y, int ldy, const void* z, int ldz, cons
 
 /* matrix_state.cu */
 long long sandy_mlstm_state_floats(int n_heads, int qk_dim, int v_dim);
+int sandy_delta_prepare_keep(const void* proj, int ld, int dtype, const float* taps, int n_taps, const float* gates, int ld_gates,
+                        const float* a_log, const float* dt_bias, float* state, long long state_stride,
+                        long long tail_off, const int* token_seq, const int* q_start, const int* seq_slots, float* qkv,
+                        int ld_qkv, float* bg, int n_tokens, int n_heads, int n_qk_heads, int qk_dim, int v_dim,
+                        float q_scale, int keep, cudaStream_t stream);
 int sandy_delta_prepare(const void* proj, int ld, int dtype, const float* taps, int n_taps, const float* gates, int ld_gates,
                         const float* a_log, const float* dt_bias, const float* state, long long state_stride,
                         long long tail_off, const int* token_seq, const int* q_start, const int* seq_slots, float* qkv,

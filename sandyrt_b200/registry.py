@@ -42,12 +42,14 @@ def _builtin_config_classes() -> Dict[str, Type[ModelConfig]]:
     from .config.panupel import PanupelConfig
     from .config.sovezen import SovezenConfig
     from .config.bilurax import BiluraxConfig
+    from .config.migelix import MigelixConfig
     from .config.pugalix import PugalixConfig
     from .config.tifepel import TifepelConfig
 
     return {GPT2Config.architecture: GPT2Config, PanupelConfig.architecture: PanupelConfig,
             SovezenConfig.architecture: SovezenConfig, BiluraxConfig.architecture: BiluraxConfig,
-            TifepelConfig.architecture: TifepelConfig, PugalixConfig.architecture: PugalixConfig}
+            TifepelConfig.architecture: TifepelConfig, PugalixConfig.architecture: PugalixConfig,
+            MigelixConfig.architecture: MigelixConfig}
 
 
 def _text(s: str) -> int:
