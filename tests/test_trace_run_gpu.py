@@ -233,3 +233,56 @@ def test_the_command_line_on_a_design_with_linear_recurrences(tmp_path):
     assert made.returncode == 0, made.stderr[-2000:]
     out = run("generate", "--model", str(tmp_path / "m"), "--dtype", "float32", "--prompt-ids", "5,17,3,9", "--max-tokens", "6")
     assert out.returncode == 0, out.stderr[-2000:]
+
+
+@pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
+def test_trace_run_serves_attention_beside_a_delta_rule(tmp_path, dtype):
+    """The same runner on a Migelix folder whose configuration leaves the ranks to the weight file: six requests
+    through four slots and a pool of 160 tokens, portions beside single tokens, a request that sits steps out.  float32
+    within 2e-4; bfloat16 within three times what rounding alone does to these requests, at least 2e-2."""
+    import plain_migelix as plain
+    from migelix_models import CONFIGS, make_weights, rel_error, write_model
+
+    cfg = CONFIGS["A"]
+    w = make_weights(cfg, seed=32)
+    model_dir = write_model(cfg, w, str(tmp_path / "model"))
+    rng = np.random.default_rng(8)
+    lengths = {"a": 60, "b": 9, "c": 33, "d": 21, "e": 30, "f": 12}
+    seqs = {k: rng.integers(0, cfg["vocab"], size=n).tolist() for k, n in lengths.items()}
+    cut = lambda k, lo, hi, want: {"id": k, "tokens": seqs[k][lo:hi], "want": want}
+    steps = [
+        {"step": 0, "entries": [cut("a", 0, 37, [36]), cut("b", 0, 2, [0, 1]), cut("c", 0, 30, [])], "end": []},
+        {"step": 1, "entries": [cut("a", 37, 38, [0]), cut("b", 2, 9, [6]), cut("d", 0, 21, [20])], "end": ["b", "d"]},
+        {"step": 2, "entries": [cut("a", 38, 60, [0, 21]), cut("e", 0, 29, [28]), cut("f", 0, 3, [2])], "end": ["a"]},
+        {"step": 3, "entries": [cut("c", 30, 31, [0]), cut("e", 29, 30, [0]), cut("f", 3, 12, [8])], "end": ["e", "f"]},
+        {"step": 4, "entries": [cut("c", 31, 33, [0, 1])], "end": ["c"]},
+    ]
+    out_dir = tmp_path / "out"
+    proc = subprocess.run([sys.executable, os.path.join(ROOT, "bin", "trace_run"), "--model", model_dir, "--dtype", dtype,
+                           "--out", str(out_dir), "--max-tokens", "160"],
+                          input="".join(json.dumps(s) + "\n" for s in steps), capture_output=True, text=True, timeout=560)
+    assert proc.returncode == 0, proc.stderr[-2000:]
+    assert [l for l in proc.stdout.splitlines() if l.startswith("done")] == [f"done {i}" for i in range(5)]
+    full = {k: plain.forward(cfg, w, v).numpy() for k, v in seqs.items()}
+    bound = 2e-4
+    if dtype == "bfloat16":
+        bound = max(2e-2, 3 * max(rel_error(plain.forward_rounded(cfg, w, v).numpy(), full[k]) for k, v in seqs.items()))
+    want = [[("a", 36), ("b", 0), ("b", 1)], [("a", 37), ("b", 8), ("d", 20)], [("a", 38), ("a", 59), ("e", 28), ("f", 2)],
+            [("c", 30), ("e", 29), ("f", 11)], [("c", 31), ("c", 32)]]
+    for i, places in enumerate(want):
+        got = np.fromfile(out_dir / f"{i}.f32", dtype="<f4").reshape(-1, cfg["vocab"])
+        assert rel_error(got, np.stack([full[k][p] for k, p in places])) < bound, f"step {i}"
+
+
+def test_the_command_line_on_attention_beside_a_delta_rule(tmp_path):
+    """`python -m sandyrt_b200 random-model` from a configuration file that states the ranks, then `generate`."""
+    from migelix_models import CONFIGS
+
+    cfg_path = tmp_path / "config.json"
+    cfg_path.write_text(json.dumps(CONFIGS["A"]))
+    run = lambda *args: subprocess.run([sys.executable, "-m", "sandyrt_b200", *args], capture_output=True, text=True, timeout=560,
+                                       cwd=ROOT)
+    made = run("random-model", "--config", str(cfg_path), "--out", str(tmp_path / "m"), "--seed", "3")
+    assert made.returncode == 0, made.stderr[-2000:]
+    out = run("generate", "--model", str(tmp_path / "m"), "--dtype", "float32", "--prompt-ids", "5,17,3,9", "--max-tokens", "6")
+    assert out.returncode == 0, out.stderr[-2000:]
