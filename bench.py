@@ -9,6 +9,7 @@
     python bench.py --capped [--chunk N]          Bilurax beside Sovezen, likewise
     python bench.py --streams [--batch B]         Tifepel beside Panupel, likewise
     python bench.py --linear [--window N]         Pugalix beside Panupel, likewise
+    python bench.py --mixing [--window N]         Migelix beside Panupel, likewise
     python bench.py --micro gemm|decode-attention|prefill-attention [...]   kernel micro-benchmarks
 
 Default workload: GPT-2 small (12 layers, width 768, 12 heads of 64, inner 3072, vocabulary 50257,
@@ -508,11 +509,28 @@ def linear_config(width, heads, kv_heads, ff, vocab=50257, layers=4, window=512)
             "layers": [{**kinds[i % 4], "mlp": {"kind": "dense", "ff": ff}} for i in range(layers)]}
 
 
+# ---- time mixing, and attention beside a delta rule with a decay per channel (Migelix) beside Panupel at equal size -------
+# Time mixing, a parallel layer, capped attention, a parallel layer in turn; heads of 64 throughout, the parallel layer's heads
+# split between its two mixers as Panupel's are; ranks of 64; a window of `window` positions; every layer with a feed-forward.
+def mixing_config(width, heads, kv_heads, ff, vocab=50257, layers=4, window=512):
+    rot = {"dims": 64, "base": 10000.0}
+    att = {"type": "attention", "mixer": {"heads": heads, "kv_heads": kv_heads, "dim": 64, "vdim": 64, "scale": 0.125, "rot": rot,
+                                          "softcap": 50.0, "mask": {"size": window}}}
+    left = {"heads": heads // 2, "kv_heads": max(kv_heads // 2, 1), "dim": 64, "vdim": 64, "scale": 0.125, "mask": {"size": window},
+            "rot": {**rot, "scaling": {"factor": 4.0, "original": 4096, "fast": 32.0, "slow": 1.0}}}
+    right = {"heads": heads // 2, "kv_heads": heads // 2, "dim": 64, "vdim": 64, "conv": 4, "rank": 64, "gate_rank": 64}
+    par = {"type": "parallel", "mixer": {"left": left, "right": right, "left_scale": 1.1, "right_scale": 0.9}}
+    wkv = {"type": "wkv", "mixer": {"heads": heads, "dim": 64, "rank": 64}}
+    kinds = [wkv, par, att, par]
+    return {"architecture": "Migelix", "vocab": vocab, "width": width, "norm": {"eps": 1e-6}, "logit_softcap": 15.0,
+            "layers": [{**kinds[i % 4], "mlp": {"kind": "dense", "ff": ff}} for i in range(layers)]}
+
+
 def hybrid(dtype_name: str, layers: int, batch: int, steps: int, warmup: int, design: str = "panupel", chunk: int = 1024,
            window: int = 512) -> int:
-    """Prefill and decode throughput of a design (Panupel, Sovezen, Bilurax, Tifepel or Pugalix) at sizes that resemble real
-    layers, beside its closest relative with the same width, heads, layer count and vocabulary (GPT-2; for Bilurax, Sovezen;
-    for Tifepel and Pugalix, Panupel),
+    """Prefill and decode throughput of a design (Panupel, Sovezen, Bilurax, Tifepel, Pugalix or Migelix) at sizes that resemble
+    real layers, beside its closest relative with the same width, heads, layer count and vocabulary (GPT-2; for Bilurax, Sovezen;
+    for Tifepel, Pugalix and Migelix, Panupel),
     both with random weights; then the device time per kernel class of both, so that like kernels can be held against
     each other.  One JSON line per size, then the tables."""
     import numpy as np
@@ -527,12 +545,13 @@ def hybrid(dtype_name: str, layers: int, batch: int, steps: int, warmup: int, de
     rng = np.random.default_rng(0)
     hybrid_config = {"panupel": globals()["hybrid_config"], "sovezen": latent_config,
                      "bilurax": lambda **kw: capped_config(chunk=chunk, **kw), "tifepel": streams_config,
-                     "pugalix": lambda **kw: linear_config(window=window, **kw)}[design]
+                     "pugalix": lambda **kw: linear_config(window=window, **kw),
+                     "migelix": lambda **kw: mixing_config(window=window, **kw)}[design]
 
     def arms(sz):
         if design == "bilurax":
             return ((design, hybrid_config(layers=layers, **sz)), ("sovezen", latent_config(layers=layers, **sz)))
-        if design in ("tifepel", "pugalix"):
+        if design in ("tifepel", "pugalix", "migelix"):
             return ((design, hybrid_config(layers=layers, **sz)), ("panupel", globals()["hybrid_config"](layers=layers, **sz)))
         gpt2_raw = {**load_model_config("small"), "n_embd": sz["width"], "n_head": sz["heads"], "n_inner": None, "n_layer": layers}
         return ((design, hybrid_config(layers=layers, **sz)), ("gpt2", gpt2_raw))
@@ -597,7 +616,10 @@ def main() -> int:
     ap.add_argument("--linear", action="store_true",
                     help="Pugalix (attention with a window that keeps the first tokens, gated linear attention, a matrix memory) "
                          "beside Panupel at equal sizes")
-    ap.add_argument("--window", type=int, default=512, help="window of --linear")
+    ap.add_argument("--mixing", action="store_true",
+                    help="Migelix (time mixing, capped attention, attention beside a delta rule with a decay per channel) beside "
+                         "Panupel at equal sizes")
+    ap.add_argument("--window", type=int, default=512, help="window of --linear and --mixing")
     ap.add_argument("--micro", nargs=argparse.REMAINDER, help="run a kernel micro-benchmark (see sandyrt_b200/csrc/microbench.py)")
     args = ap.parse_args()
     if args.impl == "reference":
@@ -608,9 +630,9 @@ def main() -> int:
     if args.micro is not None:
         from sandyrt_b200.csrc import microbench
         return microbench.main(args.micro)
-    if args.hybrid or args.latent or args.capped or args.streams or args.linear:
+    if args.hybrid or args.latent or args.capped or args.streams or args.linear or args.mixing:
         return hybrid(args.dtype, args.layers, args.batch, min(args.steps, 128), args.warmup,
-                      design="pugalix" if args.linear else "tifepel" if args.streams else "bilurax" if args.capped else
+                      design="migelix" if args.mixing else "pugalix" if args.linear else "tifepel" if args.streams else "bilurax" if args.capped else
                       "sovezen" if args.latent else "panupel", chunk=args.chunk, window=args.window)
     if args.workload:
         return workload(args.workload, args.dtype, args.layers)

@@ -65,27 +65,43 @@ __device__ __forceinline__ float log_decay(const SandyFadeRule& rule, float z, f
     return fmaxf(la, -104.0f);
 }
 
+__device__ __forceinline__ void cp16(void* smem, const void* gmem, bool valid) {
+    const unsigned dst = (unsigned)__cvta_generic_to_shared(smem);
+    const int bytes = valid ? 16 : 0;
+    asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(dst), "l"(gmem), "r"(bytes) : "memory");
+}
+
 // ---- token by token ------------------------------------------------------------------------------------------
-// Shared memory per staged token: q [d], k [d], decay [d], v [COLS], beta (delta); then the staged tokens' rows of `low` where
-// they pass tanh.
+// Shared memory per staged token: q [d], k [d], decay [d], v [COLS], beta (delta); then the staged tokens' rows of `low` [rank]; then,
+// with w_staged, the head's columns of w2t [rank][d]: weights, on their way before the kernel in front has finished.
 template <typename T, int R, int MODE>
 __global__ void __launch_bounds__(THREADS)
 fade_scan_kernel(const T* __restrict__ proj, int ld, int q_off, int k_off, int v_off, const float* __restrict__ low, int ld_low,
                  int rank, const float* __restrict__ w2t, const float* __restrict__ bias, const SandyFadeRule rule, float q_scale,
                  float* __restrict__ state, long long state_stride, const int* __restrict__ q_start,
-                 const int* __restrict__ seq_slots, float* __restrict__ out, int ld_out, int n_heads, int d, int e, int long_from) {
-    extern __shared__ float stage[];
+                 const int* __restrict__ seq_slots, float* __restrict__ out, int ld_out, int n_heads, int d, int e, int long_from,
+                 int w_staged) {
+    extern __shared__ __align__(16) float stage[];
     const int s = blockIdx.x, h = blockIdx.y, col0 = blockIdx.z * COLS;
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const int hq = h / (n_heads / rule.n_qk_heads);
     const int per = 3 * d + COLS + (MODE == DELTA ? 1 : 0);
     float* slow = stage + STAGE * per;                   // [STAGE][rank]
+    float* sw = slow + (STAGE * rank + 3) / 4 * 4;       // [rank][d]; STAGE * per is a multiple of 4
     const int t0 = q_start[s], t1 = q_start[s + 1];
     if (long_from > 0 && t1 - t0 >= long_from) {
         pdl_wait();                                      // a kernel ends only after the one before it has
         return;
     }
     float* S = state + (long long)seq_slots[s] * state_stride + (long long)h * e * d;    // [e][d]
+    if (w_staged) {
+        const int pieces = d / 4;
+        for (int x = threadIdx.x; x < rank * pieces; x += THREADS) {
+            const int r = x / pieces, i = (x % pieces) * 4;
+            cp16(sw + r * d + i, w2t + (size_t)r * n_heads * d + h * d + i, true);
+        }
+    }
+    asm volatile("cp.async.commit_group;" ::: "memory");
     const float rate = rule.decay == SANDY_DECAY_SOFTPLUS ? expf(rule.a_log[h]) : 0.0f;
     float bonus[R];
     if (MODE == BONUS)
@@ -105,21 +121,16 @@ fade_scan_kernel(const T* __restrict__ proj, int ld, int q_off, int k_off, int v
     for (int tc = t0; tc < t1; tc += STAGE) {
         const int n_tok = min(STAGE, t1 - tc);
         __syncthreads();
-        if (rule.tanh_low) {
-            for (int f = threadIdx.x; f < n_tok * rank; f += THREADS) slow[f] = tanhf(low[(size_t)(tc + f / rank) * ld_low + f % rank]);
-            __syncthreads();
+        for (int f = threadIdx.x; f < n_tok * rank; f += THREADS) {
+            const float z = low[(size_t)(tc + f / rank) * ld_low + f % rank];
+            slow[f] = rule.tanh_low ? tanhf(z) : z;
         }
         for (int f = threadIdx.x; f < n_tok * d; f += THREADS) {
-            const int tok = f / d, i = f % d, ch = h * d + i;
+            const int tok = f / d, i = f % d;
             const T* row = proj + (size_t)(tc + tok) * ld;
             float* dst = stage + tok * per;
             dst[i] = to_f32(row[q_off + hq * d + i]) * q_scale;
             dst[d + i] = to_f32(row[k_off + hq * d + i]);
-            float z = bias[ch];
-            const float* lo = rule.tanh_low ? slow + tok * rank : low + (size_t)(tc + tok) * ld_low;
-#pragma unroll 16
-            for (int r = 0; r < rank; r++) z = fmaf(w2t[(size_t)r * n_heads * d + ch], lo[r], z);
-            dst[2 * d + i] = expf(log_decay(rule, z, rate));
         }
         for (int f = threadIdx.x; f < n_tok * COLS; f += THREADS) {
             const int tok = f / COLS, c = f % COLS;
@@ -127,6 +138,22 @@ fade_scan_kernel(const T* __restrict__ proj, int ld, int q_off, int k_off, int v
         }
         if (MODE == DELTA && threadIdx.x < n_tok)
             stage[threadIdx.x * per + 3 * d + COLS] = sigmoid_f(rule.beta[(size_t)(tc + threadIdx.x) * rule.ld_beta + h]);
+        asm volatile("cp.async.wait_group 0;" ::: "memory");
+        __syncthreads();
+        for (int f = threadIdx.x; f < n_tok * d; f += THREADS) {      // the decays: rank multiplications each, in four sums
+            const int tok = f / d, i = f % d, ch = h * d + i;
+            const float* lo = slow + tok * rank;
+            const float* w = w_staged ? sw + i : w2t + ch;
+            const size_t pitch = w_staged ? d : (size_t)n_heads * d;
+            float z[4] = {bias[ch], 0.0f, 0.0f, 0.0f};
+            int r = 0;
+#pragma unroll 4
+            for (; r + 4 <= rank; r += 4)
+#pragma unroll
+                for (int c = 0; c < 4; c++) z[c] = fmaf(w[(r + c) * pitch], lo[r + c], z[c]);
+            for (; r < rank; r++) z[0] = fmaf(w[r * pitch], lo[r], z[0]);
+            stage[tok * per + 2 * d + i] = expf(log_decay(rule, (z[0] + z[1]) + (z[2] + z[3]), rate));
+        }
         __syncthreads();
         for (int tok = 0; tok < n_tok; tok++) {
             const float* in = stage + tok * per;
@@ -209,6 +236,7 @@ constexpr int CC = 32;                 // tokens per chunk
 constexpr int CT = 256;                // threads
 constexpr int PART = 8;                // tokens per part
 constexpr int PARTS = CC / PART;
+static_assert(PART == 8, "a part's tokens are two float4");
 static_assert(CT == PARTS * PART * PART, "inside the parts a thread a pair");
 
 // Place of chunk c of request s among all chunks of the step (a request brings ceil(n / CC) of them).
@@ -231,7 +259,7 @@ constexpr int LM = CC + 4;             // pitch of the triangular system's colum
 // qs, ks: float32 [T, H * dp]; P: float32 [T, H * CC]; dec: float32 [slots, H * dp]; dp = d rounded up to 4, zeros behind d.
 // Delta rule: W float32 [T, H * dp], U float32 [T, H * e].
 template <typename T, int MODE>
-__global__ void __launch_bounds__(CT)
+__global__ void __launch_bounds__(CT, MODE == DELTA ? 2 : 3)       // left alone the triangular system takes 248 registers, one block an SM
 fade_chunk_prepare_kernel(const T* __restrict__ proj, int ld, int q_off, int k_off, int v_off, const float* __restrict__ low,
                           int ld_low, int rank, const float* __restrict__ w2t, const float* __restrict__ bias,
                           const SandyFadeRule rule, float q_scale, const int* __restrict__ q_start, float* __restrict__ qs,
@@ -250,23 +278,29 @@ fade_chunk_prepare_kernel(const T* __restrict__ proj, int ld, int q_off, int k_o
     float* sk = sq + CC * lds;            // [CC][lds]
     float* sl = sk + CC * lds;            // [CC][lds]: L
     float* sp = sl + CC * lds;            // [CC][CC]
-    float* slow = sp + CC * CC;           // [CC][rank]
-    float* sbeta = slow + (CC * rank + 3) / 4 * 4;       // delta rule: [CC]
+    float* slow = sp + CC * CC;           // [rank][CC]
+    float* sbeta = slow + CC * rank;      // delta rule: [CC]
     float* sw = sbeta + CC;               // delta rule: [CC][lds], k exp(L)
     float* sm = sw + CC * lds;            // delta rule: [CC][LM], column j of the system: beta_t R(t, j), t > j
-    for (int x = tid; x < CC * dp; x += CT) {
-        const int t = x / dp, i = x % dp;
-        const bool live = t < n_tok && i < d;
-        const T* row = proj + (size_t)(tc + (live ? t : 0)) * ld;
-        sq[t * lds + i] = live ? to_f32(row[q_off + hq * d + i]) * q_scale : 0.0f;
-        sk[t * lds + i] = live ? to_f32(row[k_off + hq * d + i]) : 0.0f;
-    }
-    for (int x = tid; x < CC * rank; x += CT) {
-        const int t = x / rank, r = x % rank;
-        float z = t < n_tok ? low[(size_t)(tc + t) * ld_low + r] : 0.0f;
-        if (rule.tanh_low) z = tanhf(z);
-        slow[x] = z;
-    }
+    const int warp = tid >> 5, lane = tid & 31;
+    constexpr int NW = CT / 32;
+    for (int i = lane; i < dp; i += 32)          // a warp a row of a token, all its rows of four loads on their way at once
+#pragma unroll
+        for (int u = 0; u < CC / NW; u++) {
+            const int t = warp + u * NW;
+            const bool live = t < n_tok && i < d;
+            const T* row = proj + (size_t)(tc + (live ? t : 0)) * ld;
+            sq[t * lds + i] = live ? to_f32(row[q_off + hq * d + i]) * q_scale : 0.0f;
+            sk[t * lds + i] = live ? to_f32(row[k_off + hq * d + i]) : 0.0f;
+        }
+    for (int r = lane; r < rank; r += 32)
+#pragma unroll
+        for (int u = 0; u < CC / NW; u++) {
+            const int t = warp + u * NW;
+            float z = t < n_tok ? low[(size_t)(tc + t) * ld_low + r] : 0.0f;
+            if (rule.tanh_low) z = tanhf(z);
+            slow[r * CC + t] = z;
+        }
     for (int x = tid; x < CC * CC; x += CT) sp[x] = 0.0f;
     if (MODE == DELTA && tid < CC) sbeta[tid] = tid < n_tok ? sigmoid_f(rule.beta[(size_t)(tc + tid) * rule.ld_beta + h]) : 0.0f;
     __syncthreads();
@@ -278,10 +312,13 @@ fade_chunk_prepare_kernel(const T* __restrict__ proj, int ld, int q_off, int k_o
             const float b = bias[h * d + i];
 #pragma unroll
             for (int t = 0; t < PART; t++) z[t] = b;
+#pragma unroll 8
             for (int r = 0; r < rank; r++) {
                 const float w = w2t[(size_t)r * n_heads * d + h * d + i];
-#pragma unroll
-                for (int t = 0; t < PART; t++) z[t] = fmaf(w, slow[(part * PART + t) * rank + r], z[t]);
+                const float4 a = *reinterpret_cast<const float4*>(slow + r * CC + part * PART);
+                const float4 c4 = *reinterpret_cast<const float4*>(slow + r * CC + part * PART + 4);
+                z[0] = fmaf(w, a.x, z[0]); z[1] = fmaf(w, a.y, z[1]); z[2] = fmaf(w, a.z, z[2]); z[3] = fmaf(w, a.w, z[3]);
+                z[4] = fmaf(w, c4.x, z[4]); z[5] = fmaf(w, c4.y, z[5]); z[6] = fmaf(w, c4.z, z[6]); z[7] = fmaf(w, c4.w, z[7]);
             }
         }
         float run = 0.0f;
@@ -327,8 +364,9 @@ fade_chunk_prepare_kernel(const T* __restrict__ proj, int ld, int q_off, int k_o
         }
     }
     __syncthreads();
-    for (int x = tid; x < CC * dp; x += CT) {             // q exp(L), k exp(D - L)
-        const int t = x / dp, i = x % dp, last = (t / PART) * PART + PART - 1;
+    for (int t = warp; t < CC; t += NW)                   // q exp(L), k exp(D - L)
+    for (int i = lane; i < dp; i += 32) {
+        const int last = (t / PART) * PART + PART - 1;
         const float l = sl[t * lds + i], k = sk[t * lds + i];
         const float lq = MODE == BONUS ? (t % PART ? sl[(t - 1) * lds + i] : 0.0f) : l;
         sq[t * lds + i] *= expf(lq);
@@ -339,9 +377,9 @@ fade_chunk_prepare_kernel(const T* __restrict__ proj, int ld, int q_off, int k_o
     // pairs between parts: the keys of earlier parts fade on by one part's sum a round
     for (int p = 1; p < PARTS; p++) {
         if (p > 1) {
-            for (int x = tid; x < (p - 1) * PART * dp; x += CT) {
-                const int t = x / dp, i = x % dp;
-                sk[t * lds + i] *= expf(sl[(p * PART - 1) * lds + i]);
+            for (int i = lane; i < dp; i += 32) {         // a warp one row of every part: PART warps
+                const float f = expf(sl[(p * PART - 1) * lds + i]);
+                for (int r = 0; r < p - 1; r++) sk[(r * PART + warp) * lds + i] *= f;
             }
             __syncthreads();
         }
@@ -355,13 +393,20 @@ fade_chunk_prepare_kernel(const T* __restrict__ proj, int ld, int q_off, int k_o
     }
     // out: queries as seen from the chunk's start, keys as seen from its end, the whole chunk's fading, P
     const int ldw = n_heads * dp;
-    for (int x = tid; x < n_tok * dp; x += CT) {
-        const int t = x / dp, i = x % dp, part = t / PART;
+    static_assert(NW == PART, "a warp writes one row of every part");
+    for (int i = lane; i < dp; i += 32) {
+        const float last = expf(sl[(CC - 1) * lds + i]);
         float before = 0.0f;
-        for (int p = 0; p < part; p++) before += sl[(p * PART + PART - 1) * lds + i];
-        qs[(size_t)(tc + t) * ldw + h * dp + i] = sq[t * lds + i] * expf(before);
-        const float k = sk[t * lds + i];
-        ks[(size_t)(tc + t) * ldw + h * dp + i] = part < PARTS - 1 ? k * expf(sl[(CC - 1) * lds + i]) : k;
+#pragma unroll
+        for (int p = 0; p < PARTS; p++) {
+            const int t = p * PART + warp;
+            if (t < n_tok) {
+                qs[(size_t)(tc + t) * ldw + h * dp + i] = sq[t * lds + i] * expf(before);
+                const float k = sk[t * lds + i];
+                ks[(size_t)(tc + t) * ldw + h * dp + i] = p < PARTS - 1 ? k * last : k;
+            }
+            before += sl[(p * PART + PART - 1) * lds + i];
+        }
     }
     for (int i = tid; i < dp; i += CT) {
         float all = 0.0f;
@@ -387,7 +432,10 @@ fade_chunk_prepare_kernel(const T* __restrict__ proj, int ld, int q_off, int k_o
             } else {
                 const T* v = proj + (size_t)tc * ld + v_off + h * e + (x - dp);
 #pragma unroll
-                for (int t = 0; t < CC; t++) u[t] = t < n_tok ? sbeta[t] * to_f32(v[(size_t)t * ld]) : 0.0f;
+                for (int t = 0; t < CC; t++) {
+                    u[t] = t < n_tok ? sbeta[t] * to_f32(*v) : 0.0f;
+                    v += ld;
+                }
             }
 #pragma unroll
             for (int j = 0; j < CC - 1; j++) {
@@ -399,27 +447,23 @@ fade_chunk_prepare_kernel(const T* __restrict__ proj, int ld, int q_off, int k_o
                     if (4 * b + 2 > j) u[4 * b + 2] = fmaf(-m.z, u[j], u[4 * b + 2]);
                     u[4 * b + 3] = fmaf(-m.w, u[j], u[4 * b + 3]);
                 }
+                asm volatile("" ::: "memory");       // a column's loads stay with it: hoisted, they took every register there is
             }
             float* dst = x < dp ? W + (size_t)tc * ldw + h * dp + x : U + ((size_t)tc * n_heads + h) * e + (x - dp);
             const size_t pitch = x < dp ? (size_t)ldw : (size_t)n_heads * e;
 #pragma unroll
-            for (int t = 0; t < CC; t++)
-                if (t < n_tok) dst[t * pitch] = u[t];
+            for (int t = 0; t < CC; t++) {
+                if (t < n_tok) *dst = u[t];
+                dst += pitch;
+            }
         }
     }
     pdl_launch_dependents();
 }
 
 // ---- chunks: the recurrence ------------------------------------------------------------------------------------
-__device__ __forceinline__ void cp16(void* smem, const void* gmem, bool valid) {
-    const unsigned dst = (unsigned)__cvta_generic_to_shared(smem);
-    const int bytes = valid ? 16 : 0;
-    asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(dst), "l"(gmem), "r"(bytes) : "memory");
-}
-
-__host__ __device__ constexpr int scan_buffer_floats(int dp, bool delta) {      // q, k, P, dec, (delta) W
-    return (delta ? 3 : 2) * CC * dp + CC * CC + dp;
-}
+// q, k, P, dec, (delta) W; rows of q, k and W lie dp + 4 apart, so that a warp's four tokens meet different banks.
+__host__ __device__ constexpr int scan_buffer_floats(int dp, bool delta) { return (delta ? 3 : 2) * CC * (dp + 4) + CC * CC + dp; }
 
 // MAXR: rows of the state a thread owns (d <= 32 * MAXR).  With DELTA `proj` is U ([T, H * e], v_off 0) and a token's row of it
 // becomes u = U - W S0 before it is used.
@@ -435,8 +479,8 @@ fade_chunk_scan_kernel(const T* __restrict__ proj, int ld, int v_off, const floa
     const int t0 = q_start[s], t1 = q_start[s + 1];
     pdl_wait();
     if (t1 - t0 < long_from) return;
-    const int dp = (d + 3) / 4 * 4, ldw = n_heads * dp, buf_floats = scan_buffer_floats(dp, DELTA_RULE);
-    float* buf = smem;                              // two of (q [CC][dp], k [CC][dp], P [CC][CC], dec [dp], W [CC][dp])
+    const int dp = (d + 3) / 4 * 4, lds = dp + 4, ldw = n_heads * dp, buf_floats = scan_buffer_floats(dp, DELTA_RULE);
+    float* buf = smem;                              // two of (q [CC][lds], k [CC][lds], P [CC][CC], dec [dp], W [CC][lds])
     float* sv = buf + 2 * buf_floats;               // [CC][COLS]
     float* S0 = sv + CC * COLS;                     // [dp][COLS]
     float* S = state + (long long)seq_slots[s] * state_stride + (long long)h * e * d;
@@ -452,17 +496,17 @@ fade_chunk_scan_kernel(const T* __restrict__ proj, int ld, int v_off, const floa
             const int t = x / pieces, i = (x % pieces) * 4;
             const bool live = t < n_tok;
             const size_t at = (size_t)(live ? tc + t : t0) * ldw + h * dp + i;
-            cp16(dst + t * dp + i, qs + at, live);
-            cp16(dst + CC * dp + t * dp + i, ks + at, live);
-            if (DELTA_RULE) cp16(dst + 2 * CC * dp + CC * CC + dp + t * dp + i, W + at, live);
+            cp16(dst + t * lds + i, qs + at, live);
+            cp16(dst + CC * lds + t * lds + i, ks + at, live);
+            if (DELTA_RULE) cp16(dst + 2 * CC * lds + CC * CC + dp + t * lds + i, W + at, live);
         }
         for (int x = tid; x < CC * CC / 4; x += CT) {
             const int t = x / (CC / 4), j = (x % (CC / 4)) * 4;
             const bool live = t < n_tok;
-            cp16(dst + 2 * CC * dp + t * CC + j, P + ((size_t)(live ? tc + t : t0) * n_heads + h) * CC + j, live);
+            cp16(dst + 2 * CC * lds + t * CC + j, P + ((size_t)(live ? tc + t : t0) * n_heads + h) * CC + j, live);
         }
         for (int x = tid; x < pieces; x += CT)
-            cp16(dst + 2 * CC * dp + CC * CC + x * 4, dec + (size_t)chunk_slot(t0, s, n_tok > 0 ? (tc - t0) / CC : 0) * ldw + h * dp + x * 4, true);
+            cp16(dst + 2 * CC * lds + CC * CC + x * 4, dec + (size_t)chunk_slot(t0, s, n_tok > 0 ? (tc - t0) / CC : 0) * ldw + h * dp + x * 4, true);
         asm volatile("cp.async.commit_group;" ::: "memory");
 #pragma unroll
         for (int u = 0; u < CC * COLS / CT; u++) {
@@ -485,13 +529,13 @@ fade_chunk_scan_kernel(const T* __restrict__ proj, int ld, int v_off, const floa
         else asm volatile("cp.async.wait_group 0;" ::: "memory");
         __syncthreads();
         const float* q = buf + b * buf_floats;
-        const float* k = q + CC * dp;
-        const float* p = k + CC * dp;
+        const float* k = q + CC * lds;
+        const float* p = k + CC * lds;
         const float* fade = p + CC * CC;
         float o[2] = {0.0f, 0.0f};
         {
-            const float* qrow = q + ot * dp;
-            const float* wrow = fade + dp + ot * dp;
+            const float* qrow = q + ot * lds;
+            const float* wrow = fade + dp + ot * lds;
             float ws[2] = {0.0f, 0.0f};
 #pragma unroll 4
             for (int i = 0; i < dp; i += 4) {
@@ -550,7 +594,7 @@ fade_chunk_scan_kernel(const T* __restrict__ proj, int ld, int v_off, const floa
             for (int r = 0; r < MAXR; r++) {
                 const int i = ot + 32 * r;
                 if (i < dp) {
-                    const float x = k[j * dp + i];
+                    const float x = k[j * lds + i];
                     sn[r][0] = fmaf(x, v.x, sn[r][0]); sn[r][1] = fmaf(x, v.y, sn[r][1]);
                 }
             }
@@ -572,7 +616,7 @@ fade_chunk_scan_kernel(const T* __restrict__ proj, int ld, int v_off, const floa
 
 size_t prepare_smem(int d, int rank, bool delta) {
     const int dp = (d + 3) / 4 * 4;
-    size_t n = (size_t)3 * CC * (dp + 4) + CC * CC + (CC * rank + 3) / 4 * 4;
+    size_t n = (size_t)3 * CC * (dp + 4) + CC * CC + CC * rank;
     if (delta) n += (size_t)CC + CC * (dp + 4) + CC * LM;
     return n * sizeof(float);
 }
@@ -623,12 +667,19 @@ struct FadeCall {
 template <typename T, int MODE>
 int scan_tokens(const FadeCall& f) {
     const dim3 grid(f.n_seqs, f.n_heads, (f.e + COLS - 1) / COLS);
-    const size_t smem = (size_t)STAGE * (3 * f.d + COLS + 1 + (f.rule.tanh_low ? f.rank : 0)) * sizeof(float);
+    size_t smem = ((size_t)STAGE * (3 * f.d + COLS + 1) + (STAGE * f.rank + 3) / 4 * 4) * sizeof(float);
+    const size_t w_bytes = (size_t)f.rank * f.d * sizeof(float);
+    const int w_staged = f.d % 4 == 0 && w_bytes <= 64 * 1024 && !((uintptr_t)f.w2t & 15);
+    if (w_staged) smem += w_bytes;
 #define CASE(RR)                                                                                                         \
-    if (f.d <= 32 * RR)                                                                                                  \
+    if (f.d <= 32 * RR) {                                                                                                \
+        static size_t have = 0;                                                                                          \
+        if (int err = allow_smem(fade_scan_kernel<T, RR, MODE>, smem, have)) return err;                                 \
         return sandy_launch(fade_scan_kernel<T, RR, MODE>, grid, dim3(THREADS), smem, f.stream, (const T*)f.proj, f.ld,   \
                             f.q_off, f.k_off, f.v_off, f.low, f.ld_low, f.rank, f.w2t, f.bias, f.rule, f.q_scale, f.state, \
-                            f.state_stride, f.q_start, f.seq_slots, f.out, f.ld_out, f.n_heads, f.d, f.e, f.long_from)
+                            f.state_stride, f.q_start, f.seq_slots, f.out, f.ld_out, f.n_heads, f.d, f.e, f.long_from,    \
+                            w_staged);                                                                                   \
+    }
     CASE(1); CASE(2); CASE(3); CASE(4); CASE(6); CASE(8);
 #undef CASE
     return SANDY_ERR_UNSUPPORTED;
