@@ -364,14 +364,15 @@ fade_chunk_prepare_kernel(const T* __restrict__ proj, int ld, int q_off, int k_o
         }
     }
     __syncthreads();
-    for (int t = warp; t < CC; t += NW)                   // q exp(L), k exp(D - L)
-    for (int i = lane; i < dp; i += 32) {
+    for (int t = warp; t < CC; t += NW) {                 // q exp(L), k exp(D - L)
         const int last = (t / PART) * PART + PART - 1;
-        const float l = sl[t * lds + i], k = sk[t * lds + i];
-        const float lq = MODE == BONUS ? (t % PART ? sl[(t - 1) * lds + i] : 0.0f) : l;
-        sq[t * lds + i] *= expf(lq);
-        sk[t * lds + i] = k * expf(sl[last * lds + i] - l);
-        if (MODE == DELTA) sw[t * lds + i] = k * expf(l);
+        for (int i = lane; i < dp; i += 32) {
+            const float l = sl[t * lds + i], k = sk[t * lds + i];
+            const float lq = MODE == BONUS ? (t % PART ? sl[(t - 1) * lds + i] : 0.0f) : l;
+            sq[t * lds + i] *= expf(lq);
+            sk[t * lds + i] = k * expf(sl[last * lds + i] - l);
+            if (MODE == DELTA) sw[t * lds + i] = k * expf(l);
+        }
     }
     __syncthreads();
     // pairs between parts: the keys of earlier parts fade on by one part's sum a round

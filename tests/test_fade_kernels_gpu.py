@@ -133,7 +133,7 @@ def _att_want(case, H, Hkv, scale, window, cap, sink, gate, out_gate):
 
 
 # (H, Hkv, D, page, window, capped and gated | sinks and a factor)
-ATT = [(4, 2, 64, 16, 40, True), (12, 4, 64, 16, 0, True), (6, 2, 48, 8, 17, True), (8, 2, 128, 16, 33, True), (8, 2, 128, 16, 40, False), (16, 2, 128, 16, 0, False),
+ATT = [(4, 2, 64, 16, 40, True), (12, 4, 64, 16, 0, True), (6, 2, 48, 8, 17, True), (8, 2, 128, 16, 33, True), (10, 2, 128, 16, 45, False), (16, 2, 128, 16, 0, False),
        (4, 4, 64, 16, 70, False), (6, 3, 32, 8, 1, False), (4, 1, 128, 32, 129, False)]
 
 

@@ -273,7 +273,7 @@ ONE_LAYER = {
     "attention, one head of one entry": lambda: [layer(attention(1, 1, 1, size=7, scale=2.0), None)],
     "attention, heads of 200": lambda: [layer(attention(2, 1, 200, size=30, rot=10), None)],
     "attention, sixteen heads on one": lambda: [layer(attention(16, 1, 64, size=50, rot=16), None)],
-    "attention, heads of 128": lambda: [layer(attention(8, 2, 128, size=40, rot=64), None)],
+    "attention, heads of 128": lambda: [layer(attention(6, 2, 128, size=37, rot=48), None)],
     "left side alone": lambda: [layer(parallel(heads_of(6, 3, 32, size=13, rot=20, base=40.0, yarn=(3.0, 20, 6.0, 0.5)), delta(1, 1, 4, 4), 1.5, 0.0), None)],
     "left side alone, heads of 128, all of an entry turned": lambda: [layer(parallel(heads_of(8, 1, 128, rot=128, base=1e5, yarn=(16.0, 64, 32.0, 1.0)), delta(1, 1, 4, 4), 1.0, 0.0), None)],
     "left side alone, a ramp of no length": lambda: [layer(parallel(heads_of(2, 2, 16, rot=16, base=10.0, yarn=(2.0, 9, 3.0, 3.0)), delta(1, 1, 4, 4), 1.0, 0.0), None)],
